@@ -162,7 +162,7 @@ def inspect(model_dir: str) -> dict:
     keys = ("hidden_size", "num_hidden_layers", "num_attention_heads", "num_key_value_heads", "head_dim",
             "intermediate_size", "vocab_size", "max_position_embeddings", "rms_norm_eps", "rope_theta",
             "tie_word_embeddings", "use_sliding_window", "sliding_window", "max_window_layers", "width", "vocab", "norm", "streams",
-            "embedding")
+            "embedding", "postln_alpha")
     windows = sorted({str(layer.mixer.params.get("window")) for layer in plan.layers})
     return {"container": "safetensors", "files": len(files), "bytes": sum(os.path.getsize(f.path) for f in files),
             "tensors": len(stored), "stored_dtypes": dtypes,

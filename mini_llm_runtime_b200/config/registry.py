@@ -71,7 +71,15 @@ def config_from_dict(raw: dict):
 
 
 def config_from_dir(model_dir: str):
-    return config_from_dict(read_config_json(model_dir))
+    """The configuration of a model folder.  A config class with `with_stored_shapes(shapes)` has sizes that only the stored tensors
+    give; it gets their shapes by name, where the folder has weights."""
+    config = config_from_dict(read_config_json(model_dir))
+    if hasattr(config, "with_stored_shapes"):
+        from ..weights.safetensors_io import stored_shapes
+        shapes = stored_shapes(model_dir)
+        if shapes:
+            config = config.with_stored_shapes(shapes)
+    return config
 
 
 def plan_for(config) -> ModelPlan:

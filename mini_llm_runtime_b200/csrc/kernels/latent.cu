@@ -50,10 +50,11 @@ __global__ void __launch_bounds__(kThreads) latent_cache_kernel(const T* in, lon
 // `rot` values that all heads share as the rotated part of their keys; the cache row of a token is [latent | rotated part].  The queries'
 // own rotated parts (head h's at column q_first + h * q_step of `q`) are turned by the same angles and written behind the place of
 // that head's projected query in `qout` (column qo_first + h * qo_step).  Of the `rot` values the first `rot_dims` turn by
-// position * freq[i], float32, value 2i with value 2i + 1 (`interleaved`) or value i with value i + rot_dims / 2; the rest pass.
+// position * freq[i], float32, value 2i with value 2i + 1 (bit 0 of `layout`) or value i with value i + rot_dims / 2; the rest pass.
+// With bit 1 of `layout` one more number stands behind the frequencies: a factor on both cosine and sine.
 template <typename T>
 __global__ void __launch_bounds__(kThreads) latent_rot_cache_kernel(const T* in, long long ld, const float* weight, float eps, int rank, int rot,
-                                                                    int rot_dims, int interleaved, const float* freq, const T* q, long long ldq,
+                                                                    int rot_dims, int layout, const float* freq, const T* q, long long ldq,
                                                                     int q_first, int q_step, int heads, T* qout, long long ldqo, int qo_first,
                                                                     int qo_step, T* cache, int num_pages, const int* positions,
                                                                     const int* segment_of_row, const int* block_table, int table_stride,
@@ -64,6 +65,8 @@ __global__ void __launch_bounds__(kThreads) latent_rot_cache_kernel(const T* in,
     const int position = positions[row];
     const float p = static_cast<float>(position);
     const int half = rot_dims / 2;
+    const bool interleaved = layout & 1;
+    const float turn_mult = (layout & 2) && rot_dims ? freq[half] : 1.0f;
     // value c of a rotated part whose values are read by `at`
     auto turned = [&](auto at, int c) {
         float value = at(c);
@@ -73,6 +76,8 @@ __global__ void __launch_bounds__(kThreads) latent_rot_cache_kernel(const T* in,
             const int mate = interleaved ? c ^ 1 : (c < half ? c + half : c - half);
             float sn, cs;
             sincosf(p * freq[pair], &sn, &cs);
+            cs *= turn_mult;
+            sn *= turn_mult;
             const float other = at(mate);
             value = first ? value * cs - other * sn : value * cs + other * sn;
         }
@@ -162,10 +167,11 @@ MLR_API int mlr_latent_cache(const void* in, long long ld, int act_bf16, const v
     return mlr_launched("latent_cache");
 }
 
-// in: rows of the down projection, [rank | rot] values each (row stride ld); weight: float32 [rank]; freq: float32 [rot_dims / 2];
+// in: rows of the down projection, [rank | rot] values each (row stride ld); weight: float32 [rank]; freq: float32 [rot_dims / 2] and, with bit 1
+// of `layout`, a factor on cosine and sine behind them;
 // cache: [pages, page_size * (rank + rot)] of the activations' precision (with write_cache 0 only the queries are turned).
 MLR_API int mlr_latent_rot_cache(const void* in, long long ld, int act_bf16, const float* weight, float eps, int rank, int rot, int rot_dims,
-                                 int interleaved, const float* freq, const void* q, long long ldq, int q_first, int q_step, int heads, void* qout,
+                                 int layout, const float* freq, const void* q, long long ldq, int q_first, int q_step, int heads, void* qout,
                                  long long ldqo, int qo_first, int qo_step, void* cache, int num_pages, const int* positions,
                                  const int* segment_of_row, const int* block_table, int table_stride, int page_size, int write_cache, int rows,
                                  int* status, cudaStream_t stream) {
@@ -176,12 +182,12 @@ MLR_API int mlr_latent_rot_cache(const void* in, long long ld, int act_bf16, con
     if (rows <= 0) return 0;
     if (act_bf16)
         mlr_launch((latent_rot_cache_kernel<__nv_bfloat16>), dim3(rows), dim3(kThreads), 0, stream, static_cast<const __nv_bfloat16*>(in), ld, weight,
-                   eps, rank, rot, rot_dims, interleaved, freq, static_cast<const __nv_bfloat16*>(q), ldq, q_first, q_step, heads,
+                   eps, rank, rot, rot_dims, layout, freq, static_cast<const __nv_bfloat16*>(q), ldq, q_first, q_step, heads,
                    static_cast<__nv_bfloat16*>(qout), ldqo, qo_first, qo_step, static_cast<__nv_bfloat16*>(cache), num_pages, positions,
                    segment_of_row, block_table, table_stride, page_size, write_cache, status);
     else
         mlr_launch((latent_rot_cache_kernel<float>), dim3(rows), dim3(kThreads), 0, stream, static_cast<const float*>(in), ld, weight, eps, rank, rot,
-                   rot_dims, interleaved, freq, static_cast<const float*>(q), ldq, q_first, q_step, heads, static_cast<float*>(qout), ldqo, qo_first,
+                   rot_dims, layout, freq, static_cast<const float*>(q), ldq, q_first, q_step, heads, static_cast<float*>(qout), ldqo, qo_first,
                    qo_step, static_cast<float*>(cache), num_pages, positions, segment_of_row, block_table, table_stride, page_size, write_cache, status);
     return mlr_launched("latent_rot_cache");
 }

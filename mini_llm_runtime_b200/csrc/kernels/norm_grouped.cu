@@ -2,7 +2,8 @@
 // both what goes into a sub-layer and what comes out of it:
 //
 //   if delta:  h[row] += groupnorm(delta[row] + bias) * w_post      (the sub-layer's result, normed, joins the stream;
-//                                                                   with norm_delta = 0 it joins as it is)
+//                                                                   with norm_delta = 0 it joins as it is; with bit 2 of `norm_delta` set the SUM
+//                                                                   is normed instead: h[row] = groupnorm(h_mult * h[row] + delta[row] + bias) * w_post)
 //   if out:    out[r]  = groupnorm(h[row]) * w_pre                  (the next sub-layer's input; with bit 1 of `norm_delta`
 //                                                                   set it is h[row] itself: a sub-layer without a norm in front)
 //
@@ -71,8 +72,8 @@ constexpr int kMaxPieces = 32;
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(kThreads) group_rmsnorm_kernel(float* h, const float* delta, int ld_delta, const float* bias,
                                                                  const float* w_post, const float* w_pre, T* out, int ld_out,
-                                                                 const int* rows, int width, int groups, float eps, int mode, Pieces pieces) {
-    const int norm_delta = mode & 1, plain_out = mode & 2;
+                                                                 const int* rows, int width, int groups, float eps, int mode, float h_mult, Pieces pieces) {
+    const int norm_delta = mode & 5, plain_out = mode & 2, norm_sum = mode & 4;
     __shared__ float piece_weight[kMaxPieces];
     __shared__ long long piece_from[kMaxPieces];
     mlr_grid_wait();
@@ -126,6 +127,10 @@ __global__ void __launch_bounds__(kThreads) group_rmsnorm_kernel(float* h, const
                 const float4 b = load(bias, i);
                 v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
             }
+            if (norm_sum) {
+                const float4 old = load(hrow, i);
+                v.x = fmaf(h_mult, old.x, v.x); v.y = fmaf(h_mult, old.y, v.y); v.z = fmaf(h_mult, old.z, v.z); v.w = fmaf(h_mult, old.w, v.w);
+            }
             keep(i, v);
         }
         __syncthreads();
@@ -141,8 +146,10 @@ __global__ void __launch_bounds__(kThreads) group_rmsnorm_kernel(float* h, const
                 const float4 w = load(w_post, i);
                 v.x *= w.x; v.y *= w.y; v.z *= w.z; v.w *= w.w;
             }
-            const float4 old = load(hrow, i);
-            v.x = old.x + v.x; v.y = old.y + v.y; v.z = old.z + v.z; v.w = old.w + v.w;
+            if (!norm_sum) {
+                const float4 old = load(hrow, i);
+                v.x = old.x + v.x; v.y = old.y + v.y; v.z = old.z + v.z; v.w = old.w + v.w;
+            }
             if constexpr (VEC) *reinterpret_cast<float4*>(hrow + i) = v;
             else hrow[i] = v.x;
             keep(i, v);
@@ -181,7 +188,7 @@ __global__ void __launch_bounds__(kThreads) group_rmsnorm_kernel(float* h, const
 
 namespace {
 int group_rmsnorm(float* h, const float* delta, int ld_delta, const float* bias, const float* w_post, const float* w_pre, void* out, int ld_out,
-                  int out_bf16, const int* rows, int count, int width, int groups, float eps, int norm_delta, const Pieces& pieces,
+                  int out_bf16, const int* rows, int count, int width, int groups, float eps, int norm_delta, float h_mult, const Pieces& pieces,
                   cudaStream_t stream) {
     MLR_REQUIRE(count >= 0 && width > 0 && groups > 0 && width % groups == 0,
                 "group_rmsnorm: width %d cannot be cut into %d equal groups", width, groups);
@@ -203,7 +210,7 @@ int group_rmsnorm(float* h, const float* delta, int ld_delta, const float* bias,
         if (shared > 48 * 1024)                                                                                                        \
             cudaFuncSetAttribute(group_rmsnorm_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared)); \
         mlr_launch((group_rmsnorm_kernel<T, VEC>), dim3(count), dim3(kThreads), shared, stream, h, delta, ld_delta, bias, w_post, w_pre, \
-                   static_cast<T*>(out), ld_out, rows, width, groups, eps, norm_delta, pieces);                                       \
+                   static_cast<T*>(out), ld_out, rows, width, groups, eps, norm_delta, h_mult, pieces);                               \
     } while (0)
     if (out_bf16) {
         if (vec) MLR_NORM(__nv_bfloat16, true);
@@ -220,8 +227,18 @@ int group_rmsnorm(float* h, const float* delta, int ld_delta, const float* bias,
 MLR_API int mlr_group_rmsnorm(float* h, const float* delta, int ld_delta, const float* bias, const float* w_post,
                               const float* w_pre, void* out, int ld_out, int out_bf16, const int* rows, int count, int width,
                               int groups, float eps, int norm_delta, cudaStream_t stream) {
-    return group_rmsnorm(h, delta, ld_delta, bias, w_post, w_pre, out, ld_out, out_bf16, rows, count, width, groups, eps, norm_delta, Pieces{},
-                         stream);
+    return group_rmsnorm(h, delta, ld_delta, bias, w_post, w_pre, out, ld_out, out_bf16, rows, count, width, groups, eps, norm_delta, 1.0f,
+                         Pieces{}, stream);
+}
+
+// A norm BEHIND the sum: h[row] = groupnorm(h_mult * h[row] + delta[row] + bias) * w_post, and with `out` what the next sub-layer reads
+// of it: groupnorm(h[row]) * w_pre, or with `plain_out` h[row] itself.
+MLR_API int mlr_group_rmsnorm_sum(float* h, float h_mult, const float* delta, int ld_delta, const float* bias, const float* w_post,
+                                  const float* w_pre, void* out, int ld_out, int out_bf16, int count, int width, int groups, float eps,
+                                  int plain_out, cudaStream_t stream) {
+    MLR_REQUIRE(delta, "group_rmsnorm_sum: no contribution");
+    return group_rmsnorm(h, delta, ld_delta, bias, w_post, w_pre, out, ld_out, out_bf16, nullptr, count, width, groups, eps,
+                         4 | (plain_out ? 2 : 0), h_mult, Pieces{}, stream);
 }
 
 // The same with the contribution given in pieces (see `Pieces`): what routed experts leave, added up here instead of by a launch
@@ -233,5 +250,6 @@ MLR_API int mlr_group_rmsnorm_pieces(float* h, const float* y, long long ldy, co
                                      cudaStream_t stream) {
     MLR_REQUIRE(y, "group_rmsnorm_pieces: no pieces");
     const Pieces pieces = {y, ldy, row_of_pair, weights, top, shared_y, ld_shared, gate};
-    return group_rmsnorm(h, nullptr, 0, nullptr, w_post, w_pre, out, ld_out, out_bf16, nullptr, count, width, groups, eps, mode, pieces, stream);
+    return group_rmsnorm(h, nullptr, 0, nullptr, w_post, w_pre, out, ld_out, out_bf16, nullptr, count, width, groups, eps, mode, 1.0f, pieces,
+                         stream);
 }

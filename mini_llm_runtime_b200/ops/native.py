@@ -90,6 +90,8 @@ _SIGNATURES = {
     "norm_grouped": {
         "mlr_group_rmsnorm": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
                               c_int, c_float, c_int, c_void_p],
+        "mlr_group_rmsnorm_sum": [c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                  c_int, c_float, c_int, c_void_p],
         "mlr_group_rmsnorm_pieces": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
                                      c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
     },
@@ -113,7 +115,7 @@ _SIGNATURES = {
         "mlr_linear_recurrence": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p,
                                   c_int, c_int, c_void_p, c_void_p, c_void_p],
         "mlr_linear_recurrence_split": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p,
-                                        c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
+                                        c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
         "mlr_short_conv": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
                            c_int, c_void_p],
         "mlr_short_conv_state": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p],

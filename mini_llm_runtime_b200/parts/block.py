@@ -56,6 +56,12 @@ class SandwichBlock(Block):
     next sub-layer in the same launch.  Norm slots: "pre_mixer", "post_mixer", "pre_feed_forward",
     "post_feed_forward"; the norms must offer `emit_residual` (the grouped RMS norm does)."""
 
+    takes_pieces = True          # routed experts may leave their result in pieces for the norm behind them
+
+    def join(self, norm, b, h, result, then):
+        """The norm behind a sub-layer: its result joins the stream; returns then(stream) or None."""
+        return norm.emit_residual(b, h, result, then=then)
+
     def forward(self, h, pending, step, run):
         from ..engine.builder import EagerBuilder
         b = EagerBuilder(step)
@@ -78,21 +84,39 @@ class SandwichBlock(Block):
         if following is not None and not self.norms[last].same_shape(following):
             following = None
         if self.feed_forward is None:
-            ahead = self.norms["post_mixer"].emit_residual(b, h, mixed, then=following)
+            ahead = self.join(self.norms["post_mixer"], b, h, mixed, following)
         else:
-            x = self.norms["post_mixer"].emit_residual(b, h, mixed, then=self.norms["pre_feed_forward"])
+            x = self.join(self.norms["post_mixer"], b, h, mixed, self.norms["pre_feed_forward"])
             # A feed-forward of routed experts may leave its result in pieces for the norm behind it to add up.
-            b.accepts_pieces = bool(getattr(self.norms["post_feed_forward"], "takes_pieces", False))
+            b.accepts_pieces = self.takes_pieces and bool(getattr(self.norms["post_feed_forward"], "takes_pieces", False))
             try:
                 out = self.feed_forward.emit(b, x)
             finally:
                 b.accepts_pieces = False
-            ahead = self.norms["post_feed_forward"].emit_residual(b, h, out, then=following)
+            ahead = self.join(self.norms["post_feed_forward"], b, h, out, following)
         b.prepared = {"group_rms": following, "stream": h, "out": ahead} if following is not None else None
         return None
 
 
 register_part("block", "sandwich", SandwichBlock)
+
+
+class SumNormBlock(SandwichBlock):
+    """The norm stands behind the SUM: `h = norm(a h + mixer(h))`, then `h = norm(a h + feed_forward(h))`; a layer without a
+    feed-forward has only the first.  The stream itself is thus normed, and stays float32; the sum, the norm and the copy that
+    the next sub-layer reads (or that sub-layer's own norm) are one launch.  Parameters: alpha (a).  Norm slots as in the sandwich
+    block; a sub-layer that reads the stream as it is has an `identity` norm in front."""
+    takes_pieces = False
+
+    def __init__(self, spec, mixer, feed_forward, norms):
+        super().__init__(spec, mixer, feed_forward, norms)
+        self.alpha = float(spec.params["alpha"])
+
+    def join(self, norm, b, h, result, then):
+        return norm.emit_residual(b, h, result, then=then, sum_with=self.alpha)
+
+
+register_part("block", "sum_norm", SumNormBlock)
 
 
 class ParallelResidualBlock(Block):

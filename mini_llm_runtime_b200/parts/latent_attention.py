@@ -20,7 +20,8 @@ Further parameters, all off unless named:
                 projection has R + P rows of which the last P (not normed) are ONE rotated key part for all heads, and the score is
                 (q_plain . k_plain + q_rot . k_rot) * scale.  The cached vector of a token is [latent | rotated key part]: a key of R + P
                 values whose first R are the value.  `position` names a `rotary_frequencies` encoding (pairs side by side or halves)
-                that turns the first `dims` of the P values (`mlr_latent_rot_cache`).
+                that turns the first `dims` of the P values (`mlr_latent_rot_cache`); a scaling's factor on cosine
+                and sine is applied, to q and k alike.
     window      a query sees itself and the window - 1 tokens before it (the cache gives older pages back)
     sink        "learned": exp(sink_h) in the softmax's denominator, weight "sink" [H]
     gate        "sigmoid_head": head h's result times sigmoid((Wg x)_h), weight "g" [H, W], stacked into the first product
@@ -118,7 +119,12 @@ class LatentAttentionMixer(Mixer):
         self.w_uv_t = self.w_uv.transpose(1, 2).contiguous() if rt.is_bf16 else None
         self.latent_weight = rt.vector(tensors[w["dkv_norm"]]).float().contiguous() if self.own_latent else None
         self._sinks = rt.vector(tensors[w["sink"]]).to(device=rt.device, dtype=torch.float32).contiguous() if self.sink else None
-        self._freq = self.position.frequencies() if self.position is not None else None
+        # The frequencies, and behind them the factor on cosine and sine.
+        self._freq, self._layout = None, 0
+        if self.position is not None:
+            freq = self.position.frequencies()
+            self._freq = torch.cat([freq, torch.tensor([self.position.magnitude], dtype=torch.float32, device=freq.device)])
+            self._layout = int(self.position.interleaved) | 2
         # The rotation is done before attention (`mlr_latent_rot_cache`), so the attention kernels rotate nothing.
         self.desc = MaskedAttentionSpec(freq=None, sinks=self._sinks.data_ptr() if self.sink else None, slopes=None, heads=self.heads, kv_heads=1,
                                         dim=self.rank + self.rot, vdim=self.rank, rot_dims=0, window=self.window or 0, chunk=0,
@@ -140,7 +146,7 @@ class LatentAttentionMixer(Mixer):
             down = columns_of(proj, self._down_at, key) if self.own_latent else None
             b.launch("latent", "mlr_latent_rot_cache", down.ptr if down else None, down.ld if down else 0, proj.is_bf16,
                      self.latent_weight.data_ptr() if self.own_latent else None, self.eps, self.rank, self.rot, self.position.dims,
-                     int(self.position.interleaved), self._freq.data_ptr() if self._freq.numel() else None, proj.ptr, proj.ld, self.dim,
+                     self._layout, self._freq.data_ptr(), proj.ptr, proj.ld, self.dim,
                      self.dim + self.rot, self.heads, q.ptr, q.ld, self.rank, key, run.cache.data_ptr(), run.cache.shape[0],
                      b.meta("positions"), b.meta("segment_of_row"), b.table(run.group), b.table_stride(run.group), b.page_size,
                      int(self.own_latent), rows, b.status, b.stream)

@@ -52,6 +52,7 @@ from ..ops import functions as F
 from ..ops import native
 from ..ops.specs import GATES, QK_NORMS, MaskedAttentionSpec, address
 from .base import CacheNeed, RunContext, SequenceCore, columns_of
+from .rotary import plain_rotation
 
 
 class MaskedAttentionMixer(SequenceCore):
@@ -107,7 +108,7 @@ class MaskedAttentionMixer(SequenceCore):
 
     def attach_positions(self, positions) -> None:
         if self.position_name is not None:
-            self.position = positions[self.position_name]
+            self.position = plain_rotation(positions[self.position_name])
             if getattr(self.position, "interleaved", False):
                 raise ConfigError("the masked attention kernels pair value i with value i + dims / 2; an interleaved rotation is not built there")
             if self.position.dims > self.dim:

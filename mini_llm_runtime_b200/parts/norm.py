@@ -124,8 +124,9 @@ class GroupRmsNorm(Norm):
 
     takes_pieces = True      # `emit_residual` adds up a contribution that routed experts left in pieces (`Buf.pieces`)
 
-    def emit_residual(self, b, h, delta, then: Optional[Norm] = None):
-        """h += norm(delta + its bias) * weight; returns then(h) in the activation dtype, or None."""
+    def emit_residual(self, b, h, delta, then: Optional[Norm] = None, sum_with: Optional[float] = None):
+        """h += norm(delta + its bias) * weight; with `sum_with` = a it is the sum that is normed:
+        h = norm(a h + delta + its bias) * weight.  Returns then(h) in the activation dtype, or None."""
         if delta.slices:
             raise native.KernelError("the grouped norm takes a plain [rows, width] contribution")
         plain = isinstance(then, IdentityNorm)
@@ -139,12 +140,16 @@ class GroupRmsNorm(Norm):
         w_pre = then.weight.data_ptr() if out is not None and not plain else None
         if delta.pieces is not None:
             y, row_of_pair, weights, top, shared, gate = delta.pieces
-            if bias is not None or y.dtype is not torch.float32 or (shared is not None and shared.dtype is not torch.float32):
-                raise native.KernelError("the grouped norm adds up float32 pieces without a bias")
+            if sum_with is not None or bias is not None or y.dtype is not torch.float32 or (shared is not None and shared.dtype is not torch.float32):
+                raise native.KernelError("the grouped norm adds up float32 pieces without a bias, and not into a sum that it norms")
             b.launch("norm_grouped", "mlr_group_rmsnorm_pieces", h.ptr, y.ptr, self.width, row_of_pair.ptr, weights.ptr, top,
                      shared.ptr if shared is not None else None, shared.ld if shared is not None else 0, gate.ptr if gate is not None else None,
                      self.weight.data_ptr(), w_pre, out.ptr if out is not None else None, out.ld if out is not None else 0,
                      int(b.rt.is_bf16), h.rows, self.width, self.groups, self.eps, 1 | (2 if plain else 0), b.stream)
+        elif sum_with is not None:
+            b.launch("norm_grouped", "mlr_group_rmsnorm_sum", h.ptr, float(sum_with), delta.ptr, delta.ld,
+                     bias.data_ptr() if bias is not None else None, self.weight.data_ptr(), w_pre, out.ptr if out is not None else None,
+                     out.ld if out is not None else 0, int(b.rt.is_bf16), h.rows, self.width, self.groups, self.eps, int(plain), b.stream)
         else:
             b.launch("norm_grouped", "mlr_group_rmsnorm", h.ptr, delta.ptr, delta.ld, bias.data_ptr() if bias is not None else None,
                      self.weight.data_ptr(), w_pre, out.ptr if out is not None else None, out.ld if out is not None else 0,

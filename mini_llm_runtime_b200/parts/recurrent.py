@@ -1,6 +1,6 @@
 """Mixers with a matrix state per head and request (linear attention): retention with a fixed decay
-per head, and the gated delta rule behind short convolutions.  Both are the kernel
-`mlr_linear_recurrence` (csrc/kernels/recurrence.cu) under two descriptions.
+per head, gated linear attention with a decay per key channel, and the gated delta rule behind short convolutions with a decay per
+head or per key channel.  All are the kernel `mlr_linear_recurrence` (csrc/kernels/recurrence.cu) under different descriptions.
 
 Retention:   q, k [H, D], v [H, Dv];  q, k rotated on their first values;  k *= D^(-1/2);
              S <- decay_h S + k v^T;  o = S^T q;  o / rms(o) per head, times silu(g);  result = o Wo^T.
@@ -24,7 +24,8 @@ from ..config.registry import register_part
 from ..ops import functions as F
 from ..ops.specs import GATES, RecurrenceSpec, address
 from ..weights.loader import WeightSpec
-from .base import RunContext, SequenceCore, StateNeed, columns_of
+from .base import RunContext, SequenceCore, StateNeed
+from .rotary import plain_rotation
 
 
 def emit_recurrence(b, mixer, proj, side, act, run: RunContext) -> None:
@@ -40,13 +41,16 @@ def emit_recurrence(b, mixer, proj, side, act, run: RunContext) -> None:
                  act.ptr, act.ld, state.data_ptr(), state.stride(0), info, b.segments, proj.rows, plain.ptr if plain else None,
                  b.status, b.stream)
         return
+    # A decay per key channel, and a gate that comes of a product of small rank, are made for all rows beforehand.
+    df = b.temp(proj.rows, d.heads * d.dim, torch.float32) if d.channel_decay else None
+    gf = b.temp(proj.rows, d.heads * d.vdim, torch.float32) if d.gate_rank else None
     qf = b.temp(proj.rows, d.qk_heads * d.dim, torch.float32)
     kf = b.temp(proj.rows, d.qk_heads * d.dim, torch.float32)
     gates = b.temp(proj.rows, 2 * d.heads, torch.float32)
     obuf = b.temp(proj.rows, d.heads * d.vdim, torch.float32)
     b.launch("recurrence", "mlr_linear_recurrence_split", address(d), proj.ptr, proj.ld, side.ptr, side.ld, proj.is_bf16, act.ptr,
              act.ld, state.data_ptr(), state.stride(0), info, b.segments, b.meta("positions"), proj.rows, qf.ptr, kf.ptr, gates.ptr,
-             obuf.ptr, b.stream)
+             obuf.ptr, df.ptr if df else None, gf.ptr if gf else None, b.stream)
 
 
 def _check_state_size(dim: int, vdim: int) -> None:
@@ -77,7 +81,7 @@ class RetentionMixer(SequenceCore):
 
     def attach_positions(self, positions) -> None:
         if self.position_name is not None:
-            self.position = positions[self.position_name]
+            self.position = plain_rotation(positions[self.position_name])
             if self.position.dims > self.dim:
                 raise ConfigError(f"{self.position.dims} rotated values do not fit a head of {self.dim}")
 
@@ -159,14 +163,22 @@ class DeltaRuleMixer(SequenceCore):
         self.taps_weight = torch.cat([vec("q_conv"), vec("k_conv"), vec("v_conv")], dim=0).contiguous()
         self._held = (vec("A_log"), vec("dt_bias"), vec("norm"))
         at = self.in_columns()
+        self._held += self._channel_weights(tensors, rt)
         # q, k, v are the first columns of the projections' output and, convolved, all columns of a buffer of
         # their own; b, a and the gate are read from the projections' output.
         self.desc = RecurrenceSpec(
             a_log=self._held[0].data_ptr(), dt_bias=self._held[1].data_ptr(), out_weight=self._held[2].data_ptr(), heads=self.heads,
             qk_heads=self.qk_heads, dim=self.dim, vdim=self.vdim, prep=RecurrenceSpec.PREP["unit"], rot_dims=0,
             rule=RecurrenceSpec.RULE["delta"], gate_kind=GATES["silu"], col_q=at["q"], col_k=at["k"], col_v=at["v"],
-            col_a=at["a"], col_b=at["b"], col_gate=at["g"], q_mult=float(self.dim) ** -0.5, k_mult=1.0, unit_eps=1e-6, eps=self.eps,
+            col_a=at.get("a", 0), col_b=at["b"], col_gate=at.get("g", 0), q_mult=float(self.dim) ** -0.5, k_mult=1.0, unit_eps=1e-6, eps=self.eps,
             out_scale=float(out_scale))
+        self._describe(at)
+
+    def _channel_weights(self, tensors, rt) -> tuple:
+        return ()
+
+    def _describe(self, at) -> None:
+        """What a form of the rule changes in `desc`."""
 
     def emit_core(self, b, proj, act, run: RunContext) -> None:
         # q, k, v pass the convolutions into a buffer of their own (a row's other tokens read the
@@ -239,3 +251,117 @@ class LightningMixer(SequenceCore):
 
 
 register_part("mixer", "lightning", LightningMixer)
+
+
+RANK_LIMIT = 512
+
+
+def _check_rank(rank: int, what: str) -> int:
+    if not 1 <= rank <= RANK_LIMIT:
+        raise ConfigError(f"a {what} of rank {rank} is outside what the recurrence kernel takes (1 to {RANK_LIMIT})")
+    return rank
+
+
+def _second_half(tensors, name: str, rt) -> torch.Tensor:
+    """[rank, outputs]: the second matrix of a low-rank product as the recurrence kernels read it."""
+    return rt.matrix(tensors[name]).t().contiguous()
+
+
+class GatedLinearMixer(SequenceCore):
+    """Gated linear attention: a decay per head and key channel, made by a product of small rank.
+
+        q = Wq x D^(-1/2), k = Wk x [H, D];  v = Wv x [H, Dv];  alpha = sigmoid(A2 (A1 x) + a)^(1 / tau) [H, D]
+        S <- diag(alpha) S + k v^T;  o = S^T q;   o / rms(o) per head times a weight [Dv], times silu(Wg x);  result = o Wo^T.
+
+    Parameters: hidden_size, num_heads, head_dim, value_dim, tau, decay_rank (rows of A1), eps.  Weights: "q", "k" [H D, W],
+    "v", "g" [H Dv, W], "a1" [rank, W], "a2" [H D, rank], "a2_bias" [H D], "norm" [Dv], "o" [W, H Dv].  The state is the
+    retention mixer's: float32 [H, Dv, D] per request."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        p = spec.params
+        self.width = int(p["hidden_size"])
+        self.heads, self.dim, self.vdim = int(p["num_heads"]), int(p["head_dim"]), int(p["value_dim"])
+        self.tau, self.eps = float(p["tau"]), float(p["eps"])
+        self.rank = _check_rank(int(p["decay_rank"]), "decay")
+        if self.tau <= 0:
+            raise ConfigError(f"tau = {self.tau} must be positive")
+        _check_state_size(self.dim, self.vdim)
+        self.desc: Optional[RecurrenceSpec] = None
+
+    def state_need(self) -> StateNeed:
+        return StateNeed((self.heads * self.vdim * self.dim,), torch.float32)
+
+    def in_roles(self) -> List[Tuple[str, int]]:
+        return [("q", self.heads * self.dim), ("k", self.heads * self.dim), ("v", self.heads * self.vdim), ("g", self.heads * self.vdim),
+                ("a1", self.rank)]
+
+    def core_width(self) -> int:
+        return self.heads * self.vdim
+
+    def extra_weight_specs(self) -> List[WeightSpec]:
+        w = self.spec.weights
+        return [WeightSpec(w["a2"], (self.heads * self.dim, self.rank)),
+                WeightSpec(w["a2_bias"], (self.heads * self.dim,), "vector", ("normal", 0.5)),
+                WeightSpec(w["norm"], (self.vdim,), "vector", ("one_plus_normal", 0.01))]
+
+    def kernel_modules(self, dtype) -> List[str]:
+        return ["recurrence"] + F.product_modules(dtype)
+
+    def bind_core(self, tensors, rt, out_scale: float) -> None:
+        w = self.spec.weights
+        at = self.in_columns()
+        vec = lambda role: rt.vector(tensors[w[role]]).float().contiguous()
+        self._held = (vec("a2_bias"), vec("norm"), _second_half(tensors, w["a2"], rt))
+        self.desc = RecurrenceSpec(
+            dt_bias=self._held[0].data_ptr(), out_weight=self._held[1].data_ptr(), decay_w=self._held[2].data_ptr(), heads=self.heads,
+            qk_heads=self.heads, dim=self.dim, vdim=self.vdim, prep=RecurrenceSpec.PREP[None], rot_dims=0, rule=RecurrenceSpec.RULE["decay"],
+            gate_kind=GATES["silu"], col_q=at["q"], col_k=at["k"], col_v=at["v"], col_a=at["a1"], col_gate=at["g"],
+            channel_decay=RecurrenceSpec.CHANNEL_DECAY["sigmoid_root"], decay_rank=self.rank, q_mult=float(self.dim) ** -0.5, k_mult=1.0,
+            unit_eps=0.0, eps=self.eps, out_scale=float(out_scale), inv_tau=1.0 / self.tau)
+
+    def emit_core(self, b, proj, act, run: RunContext) -> None:
+        emit_recurrence(b, self, proj, proj, act, run)
+
+
+register_part("mixer", "gated_linear", GatedLinearMixer)
+
+
+class ChannelDeltaMixer(DeltaRuleMixer):
+    """The gated delta rule with a decay per head and key channel, and a gate that is a low-rank product through a sigmoid:
+
+        g = exp(-exp(A_log_h) softplus(A2 (A1 x) + dt_bias)) [H, D], acting on the rows of S;
+        o / rms(o) per head times a weight [Dv], times sigmoid(G2 (G1 x)).
+
+    The rest is `delta_rule`.  Further parameters: decay_rank, gate_rank (rows of A1 and G1).  Weights: "q", "k", "v", "o", "b", the three
+    convolutions, "A_log" [H] and "norm" as there, "a1" [rank, W], "a2" [H D, rank], "dt_bias" [H D], "g1" [rank, W], "g2" [H Dv, rank]."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.decay_rank = _check_rank(int(spec.params["decay_rank"]), "decay")
+        self.gate_rank = _check_rank(int(spec.params["gate_rank"]), "gate")
+
+    def in_roles(self) -> List[Tuple[str, int]]:
+        return [("q", self.qk_heads * self.dim), ("k", self.qk_heads * self.dim), ("v", self.heads * self.vdim), ("b", self.heads),
+                ("a1", self.decay_rank), ("g1", self.gate_rank)]
+
+    def extra_weight_specs(self) -> List[WeightSpec]:
+        w = self.spec.weights
+        specs = [s for s in super().extra_weight_specs() if s.name != w["dt_bias"]]
+        return specs + [WeightSpec(w["dt_bias"], (self.heads * self.dim,), "vector", ("normal", 0.5)),
+                        WeightSpec(w["a2"], (self.heads * self.dim, self.decay_rank)),
+                        WeightSpec(w["g2"], (self.heads * self.vdim, self.gate_rank))]
+
+    def _channel_weights(self, tensors, rt) -> tuple:
+        w = self.spec.weights
+        self._seconds = (_second_half(tensors, w["a2"], rt), _second_half(tensors, w["g2"], rt))
+        return self._seconds
+
+    def _describe(self, at) -> None:
+        d = self.desc
+        d.channel_decay, d.decay_rank, d.gate_rank = RecurrenceSpec.CHANNEL_DECAY["softplus"], self.decay_rank, self.gate_rank
+        d.decay_w, d.gate_w = (t.data_ptr() for t in self._seconds)
+        d.col_a, d.col_gate, d.gate_kind = at["a1"], at["g1"], GATES["sigmoid"]
+
+
+register_part("mixer", "channel_delta", ChannelDeltaMixer)

@@ -10,11 +10,13 @@ Parameters: theta, rotary_dim, max_positions.  No weights.
 """
 from __future__ import annotations
 
-from typing import Optional
+import math
+from typing import Optional, Tuple
 
 import numpy as np
 import torch
 
+from ..config.base import ConfigError
 from ..config.registry import register_part
 from .base import PositionEncoding
 
@@ -62,6 +64,19 @@ def scaled_frequencies(freq: np.ndarray, factor: float, low: float, high: float,
     return np.where(length < original / high, freq, np.where(length > original / low, freq / factor, blend))
 
 
+def yarn_frequencies(base: float, dims: int, factor: float, original: float, fast: float, slow: float) -> Tuple[np.ndarray, float]:
+    """YaRN: frequencies that turn fewer than `slow` times within `original` positions are divided by `factor`, those that turn more than
+    `fast` times stay, with a ramp over the pair index in between; and the factor 0.1 ln(factor) + 1 on every cosine and sine.
+    The pair whose frequency turns t times is dims ln(original / (2 pi t)) / (2 ln base); the ramp's ends are those of `fast`, rounded
+    down and at least 0, and of `slow`, rounded up and at most dims - 1.  float64."""
+    i = np.arange(dims // 2, dtype=np.float64)
+    freq = np.power(base, -2.0 * i / max(dims, 1))
+    pair_of = lambda turns: dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+    lo, hi = max(math.floor(pair_of(fast)), 0), min(math.ceil(pair_of(slow)), dims - 1)
+    ramp = np.clip((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return freq / factor * ramp + freq * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
 class RotaryFrequencies(PositionEncoding):
     """Rotation given as its frequencies only: `freq_i = base^(-2i/dims) / factor`, i < dims/2.  The kernels
     that use it compute `position * freq_i` and its cosine and sine in float32 themselves, so no table
@@ -69,8 +84,10 @@ class RotaryFrequencies(PositionEncoding):
     values of a head are rotated; a mixer's heads may be wider.  Value i turns with value i + dims/2, or, with
     `interleaved`, value 2i with value 2i + 1: (u, v) -> (u cos a - v sin a, v cos a + u sin a), a = position * freq_i
     (a mixer's kernels must know that layout; those that do not refuse it).
-    With `scaling` = {factor, low, high, original} only long wavelengths are slowed down (`scaled_frequencies`).
-    Parameters: base, dims, factor (default 1), interleaved (default False), scaling (default None).  No weights."""
+    With `scaling` = {factor, low, high, original} only long wavelengths are slowed down (`scaled_frequencies`); with `yarn` =
+    {factor, original, fast, slow} the frequencies are `yarn_frequencies`, and cosine and sine carry the factor `magnitude`, which a
+    mixer's kernels must apply (`plain_rotation` refuses it for those that do not).
+    Parameters: base, dims, factor (default 1), interleaved (default False), scaling, yarn (default None).  No weights."""
 
     def __init__(self, spec):
         super().__init__(spec)
@@ -85,9 +102,19 @@ class RotaryFrequencies(PositionEncoding):
         if self.scaling is not None and not (self.scaling["high"] > self.scaling["low"] and self.scaling["factor"] > 0
                                              and self.scaling["original"] > 0):
             raise ValueError(f"a frequency scaling {self.scaling} is not defined")
+        yarn = spec.params.get("yarn")
+        self.yarn = {k: float(yarn[k]) for k in ("factor", "original", "fast", "slow")} if yarn else None
+        self._yarn_freq, self.magnitude = None, 1.0
+        if self.yarn is not None:
+            if min(self.yarn.values()) <= 0 or self.base == 1.0 or self.scaling is not None or self.factor != 1.0:
+                raise ValueError(f"a YaRN scaling {self.yarn} with base {self.base} is not defined (it excludes any other scaling)")
+            self._yarn_freq, self.magnitude = yarn_frequencies(self.base, self.dims, **self.yarn)
         self._freq: Optional[torch.Tensor] = None
 
     def bind(self, tensors, rt) -> None:
+        if self._yarn_freq is not None:
+            self._freq = torch.from_numpy(self._yarn_freq.astype(np.float32)).to(rt.device)
+            return
         i = np.arange(self.dims // 2, dtype=np.float64)
         freq = np.power(self.base, -2.0 * i / max(self.dims, 1)) / self.factor
         if self.scaling is not None:
@@ -96,6 +123,13 @@ class RotaryFrequencies(PositionEncoding):
 
     def frequencies(self) -> torch.Tensor:
         return self._freq
+
+
+def plain_rotation(position):
+    """`position`, unless it needs a factor on cosine and sine that the caller's kernels do not apply."""
+    if getattr(position, "magnitude", 1.0) != 1.0:
+        raise ConfigError("this mixer rotates by plain cosines and sines: a scaling with a factor on them needs another")
+    return position
 
 
 register_part("position", "rotary_frequencies", RotaryFrequencies)

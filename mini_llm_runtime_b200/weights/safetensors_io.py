@@ -137,3 +137,14 @@ def open_model_files(model_dir: str) -> List[SafetensorsFile]:
             raise WeightFileError(f"{index} names no shard")
         return [SafetensorsFile(os.path.join(model_dir, s)) for s in shards]
     raise WeightFileError(f"{model_dir} holds neither model.safetensors nor model.safetensors.index.json")
+
+
+def stored_shapes(model_dir: str) -> Dict[str, Tuple[int, ...]]:
+    """Shape by name of every tensor a model folder stores; empty if it stores none."""
+    if not any(os.path.exists(os.path.join(model_dir, n)) for n in ("model.safetensors", "model.safetensors.index.json")):
+        return {}
+    shapes: Dict[str, Tuple[int, ...]] = {}
+    for f in open_model_files(model_dir):
+        shapes.update({name: f.shape(name) for name in f.names()})
+        f.close()
+    return shapes
