@@ -361,9 +361,26 @@ def sokolorn_config(width, ff, heads, kv, dim, layers, chunk, vocab):
     return {"architecture": "Sokolorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_softcap": 30.0, "layers": made}
 
 
-DESIGNS = {"gopevik": gopevik_config, "niridra": niridra_config, "sopetar": sopetar_config, "sokolorn": sokolorn_config}
+def gelulix_config(width, ff, heads, kv, dim, layers, chunk, vocab):
+    """A norm behind the sum of the scaled stream and each sub-layer's result.  In turn: the gated delta rule with a decay per key
+    channel (two value heads to a q/k head, a convolution of four taps, decay and gate products of rank `dim` / 2), gated linear
+    attention with a decay per key channel (rank `dim` / 2), the delta rule again, and latent attention (a cached vector of
+    3/4 `dim` values and a rotated key part of 1/4 `dim` per token, YaRN frequencies, learned sinks, no window); all with a gated
+    feed-forward with biases."""
+    mlp = {"kind": "dense", "ff": ff}
+    delta = {"heads": heads, "kv_heads": heads // 2, "dim": dim, "vdim": dim, "conv": 4, "decay_rank": dim // 2, "gate_rank": dim // 2}
+    gla = {"heads": heads, "dim": dim, "vdim": dim, "tau": 16.0, "decay_rank": dim // 2}
+    latent = {"heads": heads, "dim": dim, "rot_dim": dim // 4, "vdim": dim, "kv_rank": dim - dim // 4, "scale": (dim + dim // 4) ** -0.5,
+              "rot": {"base": 1e4, "dims": dim // 4, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    order = [("channel_delta", delta), ("gla", gla), ("channel_delta", delta), ("latent_attention", latent)]
+    return {"architecture": "Gelulix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "postln_alpha": 2.0,
+            "layers": [{"type": order[i % 4][0], "mixer": order[i % 4][1], "mlp": mlp} for i in range(layers)]}
+
+
+DESIGNS = {"gopevik": gopevik_config, "niridra": niridra_config, "sopetar": sopetar_config, "sokolorn": sokolorn_config,
+           "gelulix": gelulix_config}
 # The package's other design that stands nearest (the same attention kernels), measured as a second neighbour.
-NEIGHBOUR = {"niridra": "gopevik", "sopetar": "gopevik", "sokolorn": "sopetar"}
+NEIGHBOUR = {"niridra": "gopevik", "sopetar": "gopevik", "sokolorn": "sopetar", "gelulix": "gopevik"}
 
 
 def compare_designs(args) -> int:

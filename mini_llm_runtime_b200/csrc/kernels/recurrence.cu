@@ -31,7 +31,8 @@
 //
 // `mlr_short_conv` is the causal convolution over time per channel that precedes such a mixer in some
 // designs (taps [channels, n], the last tap is the current token's; silu after it), with the last n-1
-// inputs of every request kept as state; `mlr_short_conv_state` moves that state on after a step.
+// inputs of every request kept as state; `mlr_short_conv_state` moves that state on after a step.  `mlr_short_conv_step` does both for
+// steps of few rows.
 #include "common.cuh"
 
 #include <type_traits>
@@ -364,15 +365,56 @@ __global__ void __launch_bounds__(128) recurrence_prepare_kernel(const T* proj, 
 // read-out's gate before its sigmoid (gate_rank > 0).  A thread has one channel; the rows' small vectors stand in shared memory.
 constexpr int kChannelRows = 16, kChannelThreads = 128;
 
-template <typename T>
+// V neighbouring values as float32 (V = 1: any address; 4: an aligned group).
+template <int V, typename T>
+__device__ __forceinline__ void load_group(const T* p, float* v) {
+    if constexpr (V == 1) {
+        v[0] = mlr_load(p, 0);
+    } else if constexpr (sizeof(T) == 4) {
+#pragma unroll
+        for (int i = 0; i < V; i += 4) {
+            const float4 x = __ldcg(reinterpret_cast<const float4*>(p + i));
+            v[i] = x.x; v[i + 1] = x.y; v[i + 2] = x.z; v[i + 3] = x.w;
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < V; i += 4) {
+            const uint2 x = __ldcg(reinterpret_cast<const uint2*>(p + i));
+            const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&x.x), hi = *reinterpret_cast<const __nv_bfloat162*>(&x.y);
+            const float2 f = __bfloat1622float2(lo), g = __bfloat1622float2(hi);
+            v[i] = f.x; v[i + 1] = f.y; v[i + 2] = g.x; v[i + 3] = g.y;
+        }
+    }
+}
+
+template <int V, typename T>
+__device__ __forceinline__ void store_group(T* p, const float* v) {
+    if constexpr (V == 1) {
+        mlr_store(p, 0, v[0]);
+    } else if constexpr (sizeof(T) == 4) {
+#pragma unroll
+        for (int i = 0; i < V; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+    } else {
+#pragma unroll
+        for (int i = 0; i < V; i += 4) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(v[i], v[i + 1]), hi = __floats2bfloat162_rn(v[i + 2], v[i + 3]);
+            *reinterpret_cast<uint2*>(p + i) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        }
+    }
+}
+
+// V channels a thread (V = 4 where every row of the second matrices starts on a border of four values).
+template <typename T, int V>
 __global__ void __launch_bounds__(kChannelThreads) recurrence_channel_kernel(const T* side, int ld_side, float* df, float* gf, int rows,
                                                                              RecurrenceSpec s) {
     mlr_grid_wait();
     extern __shared__ __align__(16) float lows[];            // [rank][kChannelRows]
+    const int rank_room = s.decay_rank > s.gate_rank ? s.decay_rank : s.gate_rank;
     const int row0 = blockIdx.x * kChannelRows, n = min(kChannelRows, rows - row0);
-    const int decays = s.heads * s.dim, decay_blocks = (decays + kChannelThreads - 1) / kChannelThreads;
+    constexpr int kPerBlock = kChannelThreads * V;
+    const int decays = s.heads * s.dim, decay_blocks = (decays + kPerBlock - 1) / kPerBlock;
     const bool is_gate = static_cast<int>(blockIdx.y) >= decay_blocks;
-    const int c = (is_gate ? blockIdx.y - decay_blocks : blockIdx.y) * kChannelThreads + threadIdx.x;
+    const int c = (is_gate ? blockIdx.y - decay_blocks : blockIdx.y) * kPerBlock + threadIdx.x * V;
     const int rank = is_gate ? s.gate_rank : s.decay_rank, col = is_gate ? s.col_gate : s.col_a;
     const int width = is_gate ? s.heads * s.vdim : decays;
     for (int i = threadIdx.x; i < rank * kChannelRows; i += kChannelThreads) {
@@ -381,33 +423,54 @@ __global__ void __launch_bounds__(kChannelThreads) recurrence_channel_kernel(con
     }
     __syncthreads();
     if (c < width) {
-        const T* w = static_cast<const T*>(is_gate ? s.gate_w : s.decay_w);
-        float acc[kChannelRows] = {};
-        auto add = [&](int r, float v) {
+        const T* w = static_cast<const T*>(is_gate ? s.gate_w : s.decay_w) + c;
+        float acc[kChannelRows][V] = {};
+        auto add = [&](int r, const float* v) {
 #pragma unroll
             for (int t = 0; t < kChannelRows; t += 4) {
-                const float4 x = *reinterpret_cast<const float4*>(lows + r * kChannelRows + t);
-                acc[t] = fmaf(x.x, v, acc[t]);
-                acc[t + 1] = fmaf(x.y, v, acc[t + 1]);
-                acc[t + 2] = fmaf(x.z, v, acc[t + 2]);
-                acc[t + 3] = fmaf(x.w, v, acc[t + 3]);
+                const float4 x4 = *reinterpret_cast<const float4*>(lows + r * kChannelRows + t);
+                const float x[4] = {x4.x, x4.y, x4.z, x4.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int j = 0; j < V; ++j) acc[t + i][j] = fmaf(x[i], v[j], acc[t + i][j]);
             }
         };
+        constexpr int kAhead = 8 / V;                        // weights in flight
         int r = 0;
-        for (; r + 8 <= rank; r += 8) {
-            float v[8];
+        for (; r + kAhead <= rank; r += kAhead) {
+            float v[kAhead][V];
 #pragma unroll
-            for (int i = 0; i < 8; ++i) v[i] = mlr_load(w, static_cast<size_t>(r + i) * width + c);
+            for (int i = 0; i < kAhead; ++i) load_group<V>(w + static_cast<size_t>(r + i) * width, v[i]);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) add(r + i, v[i]);
+            for (int i = 0; i < kAhead; ++i) add(r + i, v[i]);
         }
-        for (; r < rank; ++r) add(r, mlr_load(w, static_cast<size_t>(r) * width + c));
-        float* out = (is_gate ? gf : df) + static_cast<size_t>(row0) * width + c;
-        const float bias = is_gate ? 0.0f : s.dt_bias[c];
-        const int head = is_gate ? 0 : c / s.dim;
+        for (; r < rank; ++r) {
+            float v[V];
+            load_group<V>(w + static_cast<size_t>(r) * width, v);
+            add(r, v);
+        }
+        // The decays' functions are long: they stand once, in a loop over the rows, whose sums wait in shared memory.
+        float* zs = lows + rank_room * kChannelRows + threadIdx.x * V;        // [kChannelRows][threads * V], a thread's own columns
 #pragma unroll
-        for (int t = 0; t < kChannelRows; ++t)
-            if (t < n) out[static_cast<size_t>(t) * width] = is_gate ? acc[t] : channel_decay_of(s, acc[t] + bias, head);
+        for (int t = 0; t < kChannelRows; ++t) store_group<V>(zs + t * kPerBlock, acc[t]);
+        float* out = (is_gate ? gf : df) + static_cast<size_t>(row0) * width + c;
+        float bias[V] = {};
+        if (!is_gate) {
+#pragma unroll
+            for (int j = 0; j < V; ++j) bias[j] = s.dt_bias[c + j];
+        }
+#pragma unroll 1
+        for (int t = 0; t < n; ++t) {
+            float z[V];
+#pragma unroll
+            for (int j = 0; j < V; ++j) z[j] = zs[t * kPerBlock + j];
+            if (!is_gate) {
+#pragma unroll
+                for (int j = 0; j < V; ++j) z[j] = channel_decay_of(s, z[j] + bias[j], (c + j) / s.dim);
+            }
+            store_group<V>(out + static_cast<size_t>(t) * width, z);
+        }
     }
     mlr_grid_dependents_may_start();
 }
@@ -582,84 +645,80 @@ __global__ void __launch_bounds__(kScanWarps * 32) recurrence_scan_kernel(const 
         }
 }
 
-// The same walk for head sizes that are a multiple of 32, with a warp's lanes as 4 columns x 8 lanes: a lane keeps E4 groups of
-// four state values of ONE column (values 4 * (8 * e + lane % 8) + 0..3, so that the eight lanes of a column read 128
-// consecutive bytes of k and q at a time), and a sum over a column is 3 exchanges among 8 lanes instead of 5 among 32.
-template <typename T, int E4, bool CH>
-__global__ void __launch_bounds__(kScanWarps * 32) recurrence_scan8_kernel(const float* qf, const float* kf, const float* df, const float* gates, const T* proj,
-                                                                          int ld, float* obuf, float* state, long long state_stride,
-                                                                          const int* segment_info, RecurrenceSpec s, int batch) {
+// The same walk for head sizes DIM that are a multiple of 32, with sixteen lanes a column: a lane keeps DIM / 16 state values of ONE column,
+// eight warps share the block's 16 columns (two warps a scheduler hide one another's waits).  Four tokens at a time: the sums of their
+// outputs over a column's lanes are exchanged together (five exchanges for four tokens), and nothing is stored to shared memory in
+// between; a token's k, q and decays are loaded from shared memory while the token before it is walked.
+constexpr int kColumnLanes = 16, kColumnWarps = kScanBlockCols * kColumnLanes / 32;
+
+template <typename T, int DIM, int RULE, bool CH>
+__global__ void __launch_bounds__(kColumnWarps * 32) recurrence_scan16_kernel(const float* qf, const float* kf, const float* df, const float* gates,
+                                                                            const T* proj, int ld, float* obuf, float* state, long long state_stride,
+                                                                            const int* segment_info, RecurrenceSpec s, int batch) {
     mlr_grid_wait();
+    constexpr int kThreads = kColumnWarps * 32, E = DIM / kColumnLanes, V = E % 4 == 0 ? 4 : 2;       // V: values an access
     extern __shared__ __align__(16) unsigned char smem[];
-    const size_t stage = static_cast<size_t>(batch) * s.dim;
-    float* qs = reinterpret_cast<float*>(smem);                // [2][batch][dim]: a batch is copied while the one before is walked
-    float* ks = qs + 2 * stage;                                // [2][batch][dim]
-    float* vs = ks + 2 * stage;                                // [batch][16]
-    float* os = vs + static_cast<size_t>(batch) * kScanBlockCols;   // [batch][16]
-    float* gs = os + static_cast<size_t>(batch) * kScanBlockCols;   // [batch]
+    const int stage = batch * DIM;                             // batch: a multiple of 4, at most 32
+    float* qs = reinterpret_cast<float*>(smem);                // [2][batch][DIM]: a batch is copied while the one before is walked
+    float* ks = qs + 2 * stage;                                // [2][batch][DIM]
+    float* ds = ks + 2 * stage;                                // CH: [2][batch][DIM], decays per channel
+    float* vs = ds + (CH ? 2 * stage : 0);                     // [16][batch]
+    float* os = vs + batch * kScanBlockCols;                   // [batch][16]
+    float* gs = os + batch * kScanBlockCols;                   // [batch]
     float* bs = gs + batch;                                    // [batch]
-    float* ds = gs + ((2 * batch + 3) & ~3);                   // CH: [2][batch][dim], decays per channel
-    const size_t d_ld = static_cast<size_t>(s.heads) * s.dim;
     const int segment = blockIdx.x, head = blockIdx.y, block_col = blockIdx.z * kScanBlockCols;
     const int first = segment_info[4 * segment], count = segment_info[4 * segment + 1], slot = segment_info[4 * segment + 3];
     const int qk_head = head / (s.heads / s.qk_heads);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int col0 = block_col + warp * kScanCols;
-    const size_t qk_ld = static_cast<size_t>(s.qk_heads) * s.dim;
+    const int sub = lane & (kColumnLanes - 1), my_col = warp * (32 / kColumnLanes) + lane / kColumnLanes;
+    const bool live = block_col + my_col < s.vdim;
+    const size_t qk_ld = static_cast<size_t>(s.qk_heads) * DIM, d_ld = static_cast<size_t>(s.heads) * DIM;
     const size_t o_ld = static_cast<size_t>(s.heads) * s.vdim;
-    const bool wide = s.dim % 4 == 0;                          // rows of q and k start on 16-byte borders
+    const float decay = !CH && RULE == 0 ? s.decay[head] : 1.0f;
 
-    const int sub = lane & 7, my_col = col0 + (lane >> 3);
-    const bool live = my_col < s.vdim;
-    float S[E4][4];
-    float* my_state = state + static_cast<size_t>(slot) * state_stride + (static_cast<size_t>(head) * s.vdim) * s.dim;
+    float S[E];
+    float* my_state = state + static_cast<size_t>(slot) * state_stride + (static_cast<size_t>(head) * s.vdim + block_col + my_col) * DIM;
+    // Value j of a lane is value V * (16 * (j / V) + sub) + j % V of the head: sixteen lanes read consecutive bytes.
+    auto place = [&](int j) { return V * (kColumnLanes * (j / V) + sub) + j % V; };
 #pragma unroll
-    for (int e = 0; e < E4; ++e)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) S[e][j] = live ? my_state[static_cast<size_t>(my_col) * s.dim + 4 * (8 * e + sub) + j] : 0.0f;
-    const float decay = !CH && s.rule == 0 ? s.decay[head] : 1.0f;
+    for (int j = 0; j < E; ++j) S[j] = live ? my_state[place(j)] : 0.0f;
 
-    constexpr int kVPerThread = 32 * kScanBlockCols / (kScanWarps * 32);     // batch <= 32
+    constexpr int kVPerThread = 32 * kScanBlockCols / kThreads;
     T v_next[kVPerThread];                // as loaded: a conversion right behind the load would wait for it
     float g_next = 0.0f, b_next = 0.0f;
-    // Starts the copies of a batch's q and k into a stage and loads its v, g and beta into registers.
+    // Starts the copies of a batch's q, k and decays into a stage and loads its v, g and beta into registers.
     auto fetch = [&](int base, int into) {
         const int n = min(batch, count - base);
-        const float* qsrc = qf + static_cast<size_t>(first + base) * qk_ld + static_cast<size_t>(qk_head) * s.dim;
-        const float* ksrc = kf + static_cast<size_t>(first + base) * qk_ld + static_cast<size_t>(qk_head) * s.dim;
+        const float* qsrc = qf + static_cast<size_t>(first + base) * qk_ld + static_cast<size_t>(qk_head) * DIM;
+        const float* ksrc = kf + static_cast<size_t>(first + base) * qk_ld + static_cast<size_t>(qk_head) * DIM;
+        const float* dsrc = CH ? df + static_cast<size_t>(first + base) * d_ld + static_cast<size_t>(head) * DIM : nullptr;
         float* qdst = qs + into * stage;
         float* kdst = ks + into * stage;
-        const float* dsrc = CH ? df + static_cast<size_t>(first + base) * d_ld + static_cast<size_t>(head) * s.dim : nullptr;
         float* ddst = ds + into * stage;
-        if (wide) {
-            const int per_row = s.dim / 4;
-            for (int i = threadIdx.x; i < n * per_row; i += blockDim.x) {
-                const int t = i / per_row, c = (i % per_row) * 4;
-                mlr_async_copy16(qdst + static_cast<size_t>(t) * s.dim + c, qsrc + t * qk_ld + c);
-                mlr_async_copy16(kdst + static_cast<size_t>(t) * s.dim + c, ksrc + t * qk_ld + c);
-                if constexpr (CH) mlr_async_copy16(ddst + static_cast<size_t>(t) * s.dim + c, dsrc + t * d_ld + c);
-            }
-        } else {
-            for (int i = threadIdx.x; i < n * s.dim; i += blockDim.x) {
-                const int t = i / s.dim, c = i % s.dim;
-                mlr_async_copy4(qdst + static_cast<size_t>(t) * s.dim + c, qsrc + t * qk_ld + c);
-                mlr_async_copy4(kdst + static_cast<size_t>(t) * s.dim + c, ksrc + t * qk_ld + c);
-                if constexpr (CH) mlr_async_copy4(ddst + static_cast<size_t>(t) * s.dim + c, dsrc + t * d_ld + c);
-            }
+        constexpr int kPerRow = DIM / 4;
+        for (int i = threadIdx.x; i < n * kPerRow; i += kThreads) {
+            const int t = i / kPerRow, c = (i % kPerRow) * 4;
+            mlr_async_copy16(qdst + t * DIM + c, qsrc + t * qk_ld + c);
+            mlr_async_copy16(kdst + t * DIM + c, ksrc + t * qk_ld + c);
+            if constexpr (CH) mlr_async_copy16(ddst + t * DIM + c, dsrc + t * d_ld + c);
         }
         mlr_async_commit();
 #pragma unroll
         for (int j = 0; j < kVPerThread; ++j) {
-            const int i = threadIdx.x + j * kScanWarps * 32;
+            const int i = threadIdx.x + j * kThreads;
             const int t = i / kScanBlockCols, c = block_col + i % kScanBlockCols;
             v_next[j] = proj[(t < n && c < s.vdim) ? static_cast<size_t>(first + base + t) * ld + s.col_v + head * s.vdim + c : 0];
         }
-        if (s.rule == 1 && threadIdx.x < n) {
-            if constexpr (!CH) g_next = __ldcg(gates + static_cast<size_t>(first + base + threadIdx.x) * 2 * s.heads + head);
-            b_next = __ldcg(gates + static_cast<size_t>(first + base + threadIdx.x) * 2 * s.heads + s.heads + head);
+        if (RULE == 1 && threadIdx.x < n) {
+            const float* g = gates + static_cast<size_t>(first + base + threadIdx.x) * 2 * s.heads + head;
+            if constexpr (!CH) g_next = __ldcg(g);
+            b_next = __ldcg(g + s.heads);
         }
     };
 
+    struct Token {
+        float k[E], q[E], d[CH ? E : 1];
+    };
     fetch(0, 0);
     int current = 0;
     for (int base = 0; base < count; base += batch, current ^= 1) {
@@ -667,92 +726,98 @@ __global__ void __launch_bounds__(kScanWarps * 32) recurrence_scan8_kernel(const
         __syncthreads();                    // the batch before has been walked and written out
 #pragma unroll
         for (int j = 0; j < kVPerThread; ++j) {
-            const int i = threadIdx.x + j * kScanWarps * 32;
-            if (i < batch * kScanBlockCols) vs[i] = act_in(mlr_load(&v_next[j], 0), s.in_act);
+            const int i = threadIdx.x + j * kThreads;
+            if (i < batch * kScanBlockCols) vs[i % kScanBlockCols * batch + i / kScanBlockCols] = act_in(mlr_load(&v_next[j], 0), s.in_act);
         }
-        if (threadIdx.x < batch) {
+        if (RULE == 1 && threadIdx.x < batch) {
             gs[threadIdx.x] = g_next;
             bs[threadIdx.x] = b_next;
         }
         mlr_async_wait();
         __syncthreads();
         if (base + batch < count) fetch(base + batch, current ^ 1);
-        const float* qnow = qs + current * stage;
-        const float* know = ks + current * stage;
-        const float* dnow = ds + current * stage;
-        // Four tokens at a time: their sums over a column are exchanged together, and nothing is stored to shared
-        // memory in between (a store there would keep the next token's loads from starting early).
+        const float* qnow = qs + current * stage + V * sub;
+        const float* know = ks + current * stage + V * sub;
+        const float* dnow = ds + current * stage + V * sub;
+        auto load = [&](Token& x, int t) {
+            auto vector = [&](float* into, const float* from) {
+#pragma unroll
+                for (int e = 0; e < E / V; ++e) {
+                    if constexpr (V == 4) {
+                        const float4 y = *reinterpret_cast<const float4*>(from + t * DIM + V * kColumnLanes * e);
+                        into[4 * e] = y.x; into[4 * e + 1] = y.y; into[4 * e + 2] = y.z; into[4 * e + 3] = y.w;
+                    } else {
+                        const float2 y = *reinterpret_cast<const float2*>(from + t * DIM + V * kColumnLanes * e);
+                        into[2 * e] = y.x; into[2 * e + 1] = y.y;
+                    }
+                }
+            };
+            vector(x.k, know);
+            if constexpr (CH) vector(x.d, dnow);
+            vector(x.q, qnow);
+        };
+        Token tokens[2];
+        load(tokens[0], 0);
+        // GUARDED: the batch's last, incomplete group of four.  Rows past the batch are not read: a token's successor is at most the last.
         auto walk4 = [&](int t0, auto guarded) {
+            constexpr bool kGuarded = decltype(guarded)::value;
+            const float4 v4 = *reinterpret_cast<const float4*>(vs + my_col * batch + t0);
+            const float v[4] = {v4.x, v4.y, v4.z, v4.w};
+            [[maybe_unused]] float g[4] = {decay, decay, decay, decay}, beta[4] = {};
+            if constexpr (RULE == 1) {
+                const float4 b4 = *reinterpret_cast<const float4*>(bs + t0);
+                beta[0] = b4.x; beta[1] = b4.y; beta[2] = b4.z; beta[3] = b4.w;
+                if constexpr (!CH) {
+                    const float4 g4 = *reinterpret_cast<const float4*>(gs + t0);
+                    g[0] = g4.x; g[1] = g4.y; g[2] = g4.z; g[3] = g4.w;
+                }
+            }
             float dots[4];
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
-                const int t = t0 + u;
                 dots[u] = 0.0f;
-                if (!decltype(guarded)::value || t < n) {
-                    const float4* k4 = reinterpret_cast<const float4*>(know + static_cast<size_t>(t) * s.dim);
-                    const float4* q4 = reinterpret_cast<const float4*>(qnow + static_cast<size_t>(t) * s.dim);
-                    [[maybe_unused]] const float4* d4 = reinterpret_cast<const float4*>(dnow + static_cast<size_t>(t) * s.dim);
-                    float4 kk[E4], qq[E4], dd[E4];
+                if (!kGuarded || t0 + u < n) {
+                    const Token& x = tokens[u & 1];
+                    load(tokens[(u + 1) & 1], u < 3 && !kGuarded ? t0 + u + 1 : min(t0 + u + 1, n - 1));
+                    float write = v[u];
+                    if constexpr (RULE == 0) {
 #pragma unroll
-                    for (int e = 0; e < E4; ++e) {
-                        kk[e] = k4[8 * e + sub];
-                        qq[e] = q4[8 * e + sub];
-                        if constexpr (CH) dd[e] = d4[8 * e + sub];
-                    }
-                    const float v = vs[t * kScanBlockCols + warp * kScanCols + (lane >> 3)];
-                    float d0 = 0.0f, d1 = 0.0f, d2 = 0.0f, d3 = 0.0f;
-                    if (s.rule == 0) {
-#pragma unroll
-                        for (int e = 0; e < E4; ++e) {
-                            S[e][0] = fmaf(CH ? dd[e].x : decay, S[e][0], kk[e].x * v); d0 = fmaf(S[e][0], qq[e].x, d0);
-                            S[e][1] = fmaf(CH ? dd[e].y : decay, S[e][1], kk[e].y * v); d1 = fmaf(S[e][1], qq[e].y, d1);
-                            S[e][2] = fmaf(CH ? dd[e].z : decay, S[e][2], kk[e].z * v); d2 = fmaf(S[e][2], qq[e].z, d2);
-                            S[e][3] = fmaf(CH ? dd[e].w : decay, S[e][3], kk[e].w * v); d3 = fmaf(S[e][3], qq[e].w, d3);
-                        }
+                        for (int j = 0; j < E; ++j) S[j] = fmaf(CH ? x.d[CH ? j : 0] : g[u], S[j], x.k[j] * write);
                     } else {
-                        const float g = CH ? 1.0f : gs[t], beta = bs[t];
-                        float c0 = 0.0f, c1 = 0.0f, c2 = 0.0f, c3 = 0.0f;
+                        float c[2] = {};
 #pragma unroll
-                        for (int e = 0; e < E4; ++e) {
-                            S[e][0] *= CH ? dd[e].x : g; c0 = fmaf(S[e][0], kk[e].x, c0);
-                            S[e][1] *= CH ? dd[e].y : g; c1 = fmaf(S[e][1], kk[e].y, c1);
-                            S[e][2] *= CH ? dd[e].z : g; c2 = fmaf(S[e][2], kk[e].z, c2);
-                            S[e][3] *= CH ? dd[e].w : g; c3 = fmaf(S[e][3], kk[e].w, c3);
+                        for (int j = 0; j < E; ++j) {
+                            S[j] *= CH ? x.d[CH ? j : 0] : g[u];
+                            c[j & 1] = fmaf(S[j], x.k[j], c[j & 1]);
                         }
-                        float dk = (c0 + c1) + (c2 + c3);
-                        dk += __shfl_xor_sync(0xffffffffu, dk, 1);
-                        dk += __shfl_xor_sync(0xffffffffu, dk, 2);
-                        dk += __shfl_xor_sync(0xffffffffu, dk, 4);
-                        const float u_t = beta * (v - dk);
+                        float held = c[0] + c[1];
 #pragma unroll
-                        for (int e = 0; e < E4; ++e) {
-                            S[e][0] = fmaf(kk[e].x, u_t, S[e][0]); d0 = fmaf(S[e][0], qq[e].x, d0);
-                            S[e][1] = fmaf(kk[e].y, u_t, S[e][1]); d1 = fmaf(S[e][1], qq[e].y, d1);
-                            S[e][2] = fmaf(kk[e].z, u_t, S[e][2]); d2 = fmaf(S[e][2], qq[e].z, d2);
-                            S[e][3] = fmaf(kk[e].w, u_t, S[e][3]); d3 = fmaf(S[e][3], qq[e].w, d3);
-                        }
+                        for (int step = 1; step < kColumnLanes; step *= 2) held += __shfl_xor_sync(0xffffffffu, held, step);
+                        write = beta[u] * (write - held);
+#pragma unroll
+                        for (int j = 0; j < E; ++j) S[j] = fmaf(x.k[j], write, S[j]);
                     }
-                    dots[u] = (d0 + d1) + (d2 + d3);
+                    float o[2] = {};
+#pragma unroll
+                    for (int j = 0; j < E; ++j) o[j & 1] = fmaf(S[j], x.q[j], o[j & 1]);
+                    dots[u] = o[0] + o[1];
                 }
             }
-#pragma unroll
-            for (int u = 0; u < 4; ++u) dots[u] += __shfl_xor_sync(0xffffffffu, dots[u], 1);
-#pragma unroll
-            for (int u = 0; u < 4; ++u) dots[u] += __shfl_xor_sync(0xffffffffu, dots[u], 2);
-#pragma unroll
-            for (int u = 0; u < 4; ++u) dots[u] += __shfl_xor_sync(0xffffffffu, dots[u], 4);
-            if (sub == 0) {
-#pragma unroll
-                for (int u = 0; u < 4; ++u)
-                    if (!decltype(guarded)::value || t0 + u < n) os[(t0 + u) * kScanBlockCols + warp * kScanCols + (lane >> 3)] = dots[u];
-            }
+            // Lanes with sub % 4 == u end up with the sum of token t0 + u.
+            const bool odd = sub & 1, high = sub & 2;
+            const float even_pair = (odd ? dots[1] : dots[0]) + __shfl_xor_sync(0xffffffffu, odd ? dots[0] : dots[1], 1);
+            const float odd_pair = (odd ? dots[3] : dots[2]) + __shfl_xor_sync(0xffffffffu, odd ? dots[2] : dots[3], 1);
+            float sum = (high ? odd_pair : even_pair) + __shfl_xor_sync(0xffffffffu, high ? even_pair : odd_pair, 2);
+            sum += __shfl_xor_sync(0xffffffffu, sum, 4);
+            sum += __shfl_xor_sync(0xffffffffu, sum, 8);
+            if (sub < 4 && (!kGuarded || t0 + sub < n)) os[(t0 + sub) * kScanBlockCols + my_col] = sum;
         };
         for (int t0 = 0; t0 < n; t0 += 4) {
             if (t0 + 4 <= n) walk4(t0, std::false_type{});      // whole groups carry no per-token conditions
             else walk4(t0, std::true_type{});
         }
         __syncthreads();
-        for (int i = threadIdx.x; i < n * kScanBlockCols; i += blockDim.x) {
+        for (int i = threadIdx.x; i < n * kScanBlockCols; i += kThreads) {
             const int t = i / kScanBlockCols, c = block_col + i % kScanBlockCols;
             if (c < s.vdim) obuf[static_cast<size_t>(first + base + t) * o_ld + static_cast<size_t>(head) * s.vdim + c] = os[i];
         }
@@ -760,9 +825,7 @@ __global__ void __launch_bounds__(kScanWarps * 32) recurrence_scan8_kernel(const
     mlr_grid_dependents_may_start();     // only now: blocks of the next grid that wait on this SM slow the walk
     if (live) {
 #pragma unroll
-        for (int e = 0; e < E4; ++e)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) my_state[static_cast<size_t>(my_col) * s.dim + 4 * (8 * e + sub) + j] = S[e][j];
+        for (int j = 0; j < E; ++j) my_state[place(j)] = S[j];
     }
 }
 
@@ -815,30 +878,87 @@ __global__ void __launch_bounds__(128) recurrence_readout_kernel(const float* ob
     mlr_grid_dependents_may_start();
 }
 
-template <typename T>
-__global__ void __launch_bounds__(256) short_conv_kernel(const T* in, int ld_in, T* out, int ld_out, int channels, int taps,
-                                                         const float* weights, const float* state, long long state_stride,
-                                                         const int* segment_info, const int* segment_of_row) {
+constexpr int kMaxTaps = 16;
+constexpr int kConvRows = 8, kConvThreads = 128;
+
+// A thread has V neighbouring channels and walks rows with the last taps - 1 inputs in registers.  N: the number of taps, or 0 for any
+// number (then V = 1).  STEP: a block has a segment's rows, all of them, and moves the segment's state on behind them; else it has
+// kConvRows rows of the batch, whatever their segments, and the state is read only.
+template <typename T, int V, int N, bool STEP>
+__global__ void __launch_bounds__(kConvThreads) short_conv_kernel(const T* in, int ld_in, T* out, int ld_out, int channels, int taps,
+                                                                  const float* weights, float* state, long long state_stride,
+                                                                  const int* segment_info, const int* segment_of_row, int rows) {
     mlr_grid_wait();
-    const int row = blockIdx.x;
-    const int segment = segment_of_row[row];
-    const int first = segment_info[4 * segment], slot = segment_info[4 * segment + 3];
-    const int j = row - first;
-    const float* old = state + static_cast<size_t>(slot) * state_stride;
-    for (int c = threadIdx.x; c < channels; c += blockDim.x) {
-        float y = 0.0f;
-        for (int i = 0; i < taps; ++i) {
-            const int m = j - (taps - 1) + i;      // the input this tap sees, counted from the step's first token
-            const float x = m >= 0 ? mlr_load(in + static_cast<size_t>(first + m) * ld_in, c)
-                                   : old[static_cast<size_t>(taps - 1 + m) * channels + c];
-            y = fmaf(weights[static_cast<size_t>(c) * taps + i], x, y);
+    constexpr int kBack = (N ? N : kMaxTaps) - 1;
+    const int back = N ? N - 1 : taps - 1;
+    const int c = (blockIdx.y * kConvThreads + threadIdx.x) * V;
+    if (c >= channels) return;
+    float w[kBack + 1][V], past[kBack + 1][V];                  // past[i]: the input that tap i sees
+#pragma unroll
+    for (int i = 0; i <= kBack; ++i)
+#pragma unroll
+        for (int j = 0; j < V; ++j) w[i][j] = i <= back ? weights[static_cast<size_t>(c + j) * (back + 1) + i] : 0.0f;
+    int row = STEP ? segment_info[4 * blockIdx.x] : blockIdx.x * kConvRows;
+    const int end = STEP ? row + segment_info[4 * blockIdx.x + 1] : min(row + kConvRows, rows);
+    int segment = -1;
+    float next[V];
+    if (row < end) load_group<V>(in + static_cast<size_t>(row) * ld_in + c, next);
+    float* mine = nullptr;
+    for (; row < end; ++row) {
+        const int now = STEP ? static_cast<int>(blockIdx.x) : segment_of_row[row];
+        if (now != segment) {                                   // the inputs before this row: of this step, or from the state
+            segment = now;
+            const int first = segment_info[4 * segment], j0 = row - first;
+            mine = state + static_cast<size_t>(segment_info[4 * segment + 3]) * state_stride + c;
+#pragma unroll
+            for (int i = 0; i < kBack; ++i)
+                if (i < back) {
+                    const int m = j0 - back + i;
+                    if (m >= 0) load_group<V>(in + static_cast<size_t>(first + m) * ld_in + c, past[i]);
+                    else {
+#pragma unroll
+                        for (int j = 0; j < V; ++j) past[i][j] = mine[static_cast<size_t>(back + m) * channels + j];
+                    }
+                }
         }
-        mlr_store(out + static_cast<size_t>(row) * ld_out, c, y / (1.0f + expf(-y)));
+        float x[V], y[V] = {};
+#pragma unroll
+        for (int j = 0; j < V; ++j) x[j] = next[j];
+        if (row + 1 < end) load_group<V>(in + static_cast<size_t>(row + 1) * ld_in + c, next);
+#pragma unroll
+        for (int i = 0; i < kBack; ++i)
+            if (i < back) {
+#pragma unroll
+                for (int j = 0; j < V; ++j) y[j] = fmaf(w[i][j], past[i][j], y[j]);
+            }
+#pragma unroll
+        for (int i = 0; i <= kBack; ++i)
+            if (i == back) {
+#pragma unroll
+                for (int j = 0; j < V; ++j) y[j] = fmaf(w[i][j], x[j], y[j]);
+            }
+#pragma unroll
+        for (int j = 0; j < V; ++j) y[j] = y[j] / (1.0f + expf(-y[j]));
+        store_group<V>(out + static_cast<size_t>(row) * ld_out + c, y);
+#pragma unroll
+        for (int i = 0; i < kBack; ++i)
+            if (i < back) {
+#pragma unroll
+                for (int j = 0; j < V; ++j) past[i][j] = i + 1 < back ? past[i + 1][j] : x[j];
+            }
+    }
+    if constexpr (STEP) {
+        if (mine) {
+#pragma unroll
+            for (int i = 0; i < kBack; ++i)
+                if (i < back) {
+#pragma unroll
+                    for (int j = 0; j < V; ++j) mine[static_cast<size_t>(i) * channels + j] = past[i][j];
+                }
+        }
     }
     mlr_grid_dependents_may_start();
 }
-
-constexpr int kMaxTaps = 16;
 
 template <typename T>
 __global__ void __launch_bounds__(256) short_conv_state_kernel(const T* in, int ld_in, int channels, int taps, float* state,
@@ -962,37 +1082,49 @@ MLR_API int mlr_linear_recurrence_split(const RecurrenceSpec* spec, const void* 
     const size_t per_token = sizeof(float) * ((channel ? 6 : 4) * static_cast<size_t>(s.dim) + 2 * kScanBlockCols + 2);
     int batch = static_cast<int>(((channel ? 84 : 44) * 1024) / per_token);
     batch = batch < 1 ? 1 : (batch > 32 ? 32 : batch);
+    if (batch > 4) batch -= batch % 4;
     const size_t shared = per_token * batch + (channel ? 16 : 0);
     const dim3 grid(n_segments, s.heads, (s.vdim + kScanBlockCols - 1) / kScanBlockCols);
+    const int group = s.heads * s.dim % 4 == 0 && s.heads * s.vdim % 4 == 0 ? 4 : 1;       // channels a thread of the channel kernel
+    const int per_block = kChannelThreads * group;
     const dim3 channel_grid((rows + kChannelRows - 1) / kChannelRows,
-                            (s.heads * s.dim + kChannelThreads - 1) / kChannelThreads +
-                                (s.gate_rank ? (s.heads * s.vdim + kChannelThreads - 1) / kChannelThreads : 0));
-    const size_t channel_shared = sizeof(float) * kChannelRows * static_cast<size_t>(s.decay_rank > s.gate_rank ? s.decay_rank : s.gate_rank);
-#define MLR_WALK(KERNEL, T)                                                                                                            \
+                            (s.heads * s.dim + per_block - 1) / per_block + (s.gate_rank ? (s.heads * s.vdim + per_block - 1) / per_block : 0));
+    const size_t channel_shared = sizeof(float) * kChannelRows * (static_cast<size_t>(s.decay_rank > s.gate_rank ? s.decay_rank : s.gate_rank) + per_block);
+#define MLR_WALK(KERNEL, T, WARPS)                                                                                                     \
     do {                                                                                                                               \
         if (shared > 48 * 1024) cudaFuncSetAttribute(KERNEL, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));   \
-        mlr_launch((KERNEL), dim3(grid), dim3(kScanWarps * 32), shared, stream, qf, kf, static_cast<const float*>(df), gates,          \
+        mlr_launch((KERNEL), dim3(grid), dim3((WARPS) * 32), shared, stream, qf, kf, static_cast<const float*>(df), gates,             \
                    static_cast<const T*>(proj), ld, obuf, state, state_stride, segment_info, s, batch);                                \
+    } while (0)
+#define MLR_COLUMN(T, DIM, CH)                                                                                                         \
+    do {                                                                                                                               \
+        if (s.rule == 0) MLR_WALK((recurrence_scan16_kernel<T, DIM, 0, CH>), T, kColumnWarps);                                         \
+        else MLR_WALK((recurrence_scan16_kernel<T, DIM, 1, CH>), T, kColumnWarps);                                                     \
     } while (0)
 #define MLR_SCAN(T, CH)                                                                                                                \
     do {                                                                                                                               \
-        if (s.dim == 32) MLR_WALK((recurrence_scan8_kernel<T, 1, CH>), T);                                                             \
-        else if (s.dim == 64) MLR_WALK((recurrence_scan8_kernel<T, 2, CH>), T);                                                        \
-        else if (s.dim == 96) MLR_WALK((recurrence_scan8_kernel<T, 3, CH>), T);                                                        \
-        else if (s.dim == 128) MLR_WALK((recurrence_scan8_kernel<T, 4, CH>), T);                                                       \
-        else if (s.dim == 256) MLR_WALK((recurrence_scan8_kernel<T, 8, CH>), T);                                                       \
-        else if (regs == 1) MLR_WALK((recurrence_scan_kernel<T, 1, CH>), T);                                                           \
-        else if (regs == 2) MLR_WALK((recurrence_scan_kernel<T, 2, CH>), T);                                                           \
-        else if (regs == 4) MLR_WALK((recurrence_scan_kernel<T, 4, CH>), T);                                                           \
-        else MLR_WALK((recurrence_scan_kernel<T, 8, CH>), T);                                                                          \
+        if (s.dim == 32) MLR_COLUMN(T, 32, CH);                                                                                        \
+        else if (s.dim == 64) MLR_COLUMN(T, 64, CH);                                                                                   \
+        else if (s.dim == 96) MLR_COLUMN(T, 96, CH);                                                                                   \
+        else if (s.dim == 128) MLR_COLUMN(T, 128, CH);                                                                                 \
+        else if (s.dim == 256) MLR_COLUMN(T, 256, CH);                                                                                 \
+        else if (regs == 1) MLR_WALK((recurrence_scan_kernel<T, 1, CH>), T, kScanWarps);                                               \
+        else if (regs == 2) MLR_WALK((recurrence_scan_kernel<T, 2, CH>), T, kScanWarps);                                               \
+        else if (regs == 4) MLR_WALK((recurrence_scan_kernel<T, 4, CH>), T, kScanWarps);                                               \
+        else MLR_WALK((recurrence_scan_kernel<T, 8, CH>), T, kScanWarps);                                                              \
     } while (0)
 #define MLR_SPLIT(T)                                                                                                                   \
     do {                                                                                                                               \
         mlr_launch((recurrence_prepare_kernel<T>), dim3(rows), dim3(128), 0, stream, static_cast<const T*>(proj), ld,                  \
                    static_cast<const T*>(side), ld_side, qf, kf, gates, positions, s);                                                 \
         if (channel) {                                                                                                                 \
-            mlr_launch((recurrence_channel_kernel<T>), dim3(channel_grid), dim3(kChannelThreads), channel_shared, stream,              \
-                       static_cast<const T*>(side), ld_side, df, gf, rows, s);                                                         \
+            if (channel_shared > 48 * 1024)                                                                                            \
+                cudaFuncSetAttribute(group == 4 ? recurrence_channel_kernel<T, 4> : recurrence_channel_kernel<T, 1>,                   \
+                                     cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(channel_shared));                   \
+            if (group == 4) mlr_launch((recurrence_channel_kernel<T, 4>), dim3(channel_grid), dim3(kChannelThreads), channel_shared,   \
+                                       stream, static_cast<const T*>(side), ld_side, df, gf, rows, s);                                 \
+            else mlr_launch((recurrence_channel_kernel<T, 1>), dim3(channel_grid), dim3(kChannelThreads), channel_shared, stream,      \
+                            static_cast<const T*>(side), ld_side, df, gf, rows, s);                                                    \
             MLR_SCAN(T, true);                                                                                                         \
         } else {                                                                                                                       \
             MLR_SCAN(T, false);                                                                                                        \
@@ -1004,9 +1136,37 @@ MLR_API int mlr_linear_recurrence_split(const RecurrenceSpec* spec, const void* 
     else MLR_SPLIT(float);
 #undef MLR_SPLIT
 #undef MLR_SCAN
+#undef MLR_COLUMN
 #undef MLR_WALK
     return mlr_launched("linear_recurrence_split");
 }
+
+namespace {
+template <bool STEP>
+int short_conv(const void* in, int ld_in, void* out, int ld_out, int act_bf16, int channels, int taps, const float* weights, float* state,
+               long long state_stride, const int* segment_info, const int* segment_of_row, int blocks, int rows, cudaStream_t stream) {
+    const size_t group_bytes = act_bf16 ? 8 : 16;
+    const bool wide = taps <= 4 && channels % 4 == 0 && ld_in % 4 == 0 && ld_out % 4 == 0 && reinterpret_cast<uintptr_t>(in) % group_bytes == 0 &&
+                      reinterpret_cast<uintptr_t>(out) % group_bytes == 0;
+    const dim3 grid(blocks, (channels + kConvThreads * (wide ? 4 : 1) - 1) / (kConvThreads * (wide ? 4 : 1)));
+#define MLR_CONV(T, V, N)                                                                                                              \
+    mlr_launch((short_conv_kernel<T, V, N, STEP>), dim3(grid), dim3(kConvThreads), 0, stream, static_cast<const T*>(in), ld_in,        \
+               static_cast<T*>(out), ld_out, channels, taps, weights, state, state_stride, segment_info, segment_of_row, rows)
+#define MLR_CONVS(T)                                                                                                                   \
+    do {                                                                                                                               \
+        if (!wide) MLR_CONV(T, 1, 0);                                                                                                  \
+        else if (taps == 1) MLR_CONV(T, 4, 1);                                                                                         \
+        else if (taps == 2) MLR_CONV(T, 4, 2);                                                                                         \
+        else if (taps == 3) MLR_CONV(T, 4, 3);                                                                                         \
+        else MLR_CONV(T, 4, 4);                                                                                                        \
+    } while (0)
+    if (act_bf16) MLR_CONVS(__nv_bfloat16);
+    else MLR_CONVS(float);
+#undef MLR_CONVS
+#undef MLR_CONV
+    return mlr_launched("short_conv");
+}
+}  // namespace
 
 MLR_API int mlr_short_conv(const void* in, int ld_in, void* out, int ld_out, int act_bf16, int channels, int taps,
                            const float* weights, const float* state, long long state_stride, const int* segment_info,
@@ -1014,13 +1174,18 @@ MLR_API int mlr_short_conv(const void* in, int ld_in, void* out, int ld_out, int
     MLR_REQUIRE(channels > 0 && taps >= 1 && taps <= kMaxTaps, "short_conv: %d taps are outside [1, %d]", taps, kMaxTaps);
     MLR_REQUIRE(ld_in >= channels && ld_out >= channels && (taps == 1 || state), "short_conv: bad strides or no state");
     if (rows <= 0) return 0;
-    if (act_bf16)
-        mlr_launch((short_conv_kernel<__nv_bfloat16>), dim3(rows), dim3(256), 0, stream, static_cast<const __nv_bfloat16*>(in), ld_in,
-                   static_cast<__nv_bfloat16*>(out), ld_out, channels, taps, weights, state, state_stride, segment_info, segment_of_row);
-    else
-        mlr_launch((short_conv_kernel<float>), dim3(rows), dim3(256), 0, stream, static_cast<const float*>(in), ld_in,
-                   static_cast<float*>(out), ld_out, channels, taps, weights, state, state_stride, segment_info, segment_of_row);
-    return mlr_launched("short_conv");
+    return short_conv<false>(in, ld_in, out, ld_out, act_bf16, channels, taps, weights, const_cast<float*>(state), state_stride, segment_info,
+                             segment_of_row, (rows + kConvRows - 1) / kConvRows, rows, stream);
+}
+
+// The convolution and the state behind it in one launch: a block walks all rows of a segment (steps of few rows).
+MLR_API int mlr_short_conv_step(const void* in, int ld_in, void* out, int ld_out, int act_bf16, int channels, int taps, const float* weights,
+                                float* state, long long state_stride, const int* segment_info, int n_segments, cudaStream_t stream) {
+    MLR_REQUIRE(channels > 0 && taps >= 1 && taps <= kMaxTaps, "short_conv_step: %d taps are outside [1, %d]", taps, kMaxTaps);
+    MLR_REQUIRE(ld_in >= channels && ld_out >= channels && (taps == 1 || state), "short_conv_step: bad strides or no state");
+    if (n_segments <= 0) return 0;
+    return short_conv<true>(in, ld_in, out, ld_out, act_bf16, channels, taps, weights, state, state_stride, segment_info, nullptr, n_segments, 0,
+                            stream);
 }
 
 MLR_API int mlr_short_conv_state(const void* in, int ld_in, int act_bf16, int channels, int taps, float* state,

@@ -189,10 +189,14 @@ class DeltaRuleMixer(SequenceCore):
         stride = state.stride(0)
         info, of_row = b.meta("segment_info"), b.meta("segment_of_row")
         conv = b.temp(proj.rows, self.channels, proj.dtype)
-        b.launch("recurrence", "mlr_short_conv", proj.ptr, proj.ld, conv.ptr, conv.ld, proj.is_bf16, self.channels, self.taps,
-                 self.taps_weight.data_ptr(), conv_state, stride, info, of_row, proj.rows, b.stream)
-        b.launch("recurrence", "mlr_short_conv_state", proj.ptr, proj.ld, proj.is_bf16, self.channels, self.taps, conv_state, stride,
-                 info, b.segments, b.stream)
+        if b.le(proj.rows, b.rt.recurrence_fused_rows):
+            b.launch("recurrence", "mlr_short_conv_step", proj.ptr, proj.ld, conv.ptr, conv.ld, proj.is_bf16, self.channels, self.taps,
+                     self.taps_weight.data_ptr(), conv_state, stride, info, b.segments, b.stream)
+        else:
+            b.launch("recurrence", "mlr_short_conv", proj.ptr, proj.ld, conv.ptr, conv.ld, proj.is_bf16, self.channels, self.taps,
+                     self.taps_weight.data_ptr(), conv_state, stride, info, of_row, proj.rows, b.stream)
+            b.launch("recurrence", "mlr_short_conv_state", proj.ptr, proj.ld, proj.is_bf16, self.channels, self.taps, conv_state, stride,
+                     info, b.segments, b.stream)
         emit_recurrence(b, self, conv, proj, act, run)
 
 
