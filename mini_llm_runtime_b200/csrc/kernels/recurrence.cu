@@ -832,10 +832,14 @@ __global__ void __launch_bounds__(kColumnWarps * 32) recurrence_scan16_kernel(co
 
 // Norm per head, weight, gate and the constant on the scan's float32 outputs [rows, heads * vdim].  gf: the gate's values in
 // float32 [rows, heads * vdim] when they come of a low-rank product, else null and the gate is in `side`.
-template <typename T>
-__global__ void __launch_bounds__(128) recurrence_readout_kernel(const float* obuf, const T* side, int ld_side, const float* gf, T* out,
-                                                                 int ld_out, RecurrenceSpec s) {
+// VEC: four values an access, a head's values held in registers between the sum and the result (vdim a multiple of 4, at most 256).
+constexpr int kReadoutThreads = 256;
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kReadoutThreads) recurrence_readout_kernel(const float* obuf, const T* side, int ld_side, const float* gf, T* out,
+                                                                            int ld_out, RecurrenceSpec s) {
     mlr_grid_wait();
+    constexpr int V = VEC ? 4 : 1, kHeld = 256 / (32 * V);
     const int row = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     __shared__ float scratch[32];
@@ -852,27 +856,47 @@ __global__ void __launch_bounds__(128) recurrence_readout_kernel(const float* ob
     }
     for (int head = warp; head < s.heads; head += warps) {
         const float* o = obuf + (static_cast<size_t>(row) * s.heads + head) * s.vdim;
+        float held[kHeld][V];
+#pragma unroll
+        for (int i = 0; i < kHeld; ++i) {
+            const int c = (i * 32 + lane) * V;
+            if (c < s.vdim) load_group<V>(o + c, held[i]);
+        }
         float inv = inv_all;
         if (s.eps >= 0.0f && !s.norm_all) {
             float sum = 0.0f;
-            for (int c = lane; c < s.vdim; c += 32) {
-                const float v = __ldcg(o + c);
-                sum = fmaf(v, v, sum);
-            }
+#pragma unroll
+            for (int i = 0; i < kHeld; ++i)
+                if ((i * 32 + lane) * V < s.vdim) {
+#pragma unroll
+                    for (int j = 0; j < V; ++j) sum = fmaf(held[i][j], held[i][j], sum);
+                }
             inv = 1.0f / sqrtf(mlr_warp_sum(sum) / static_cast<float>(s.vdim) + s.eps);
         }
-        const T* grow = side + static_cast<size_t>(row) * ld_side;
+        const T* grow = side + static_cast<size_t>(row) * ld_side + s.col_gate + head * s.vdim;
+        const float* gfrow = gf + (static_cast<size_t>(row) * s.heads + head) * s.vdim;
         T* orow = out + static_cast<size_t>(row) * ld_out + static_cast<size_t>(head) * s.vdim;
-        for (int c = lane; c < s.vdim; c += 32) {
-            float value = __ldcg(o + c) * inv;
-            if (s.out_weight) value *= s.out_weight[s.norm_all ? head * s.vdim + c : c];
+#pragma unroll
+        for (int i = 0; i < kHeld; ++i) {
+            const int c = (i * 32 + lane) * V;
+            if (c >= s.vdim) break;
+            float g[V] = {};
             if (s.gate_kind) {
-                const float g = gf ? __ldcg(gf + (static_cast<size_t>(row) * s.heads + head) * s.vdim + c)
-                                   : mlr_load(grow, s.col_gate + head * s.vdim + c);
-                const float sig = 1.0f / (1.0f + expf(-g));
-                value *= s.gate_kind == 2 ? g * sig : sig;
+                if (gf) load_group<V>(gfrow + c, g);
+                else load_group<V>(grow + c, g);
             }
-            mlr_store(orow, c, value * s.out_scale);
+            float value[V];
+#pragma unroll
+            for (int j = 0; j < V; ++j) {
+                value[j] = held[i][j] * inv;
+                if (s.out_weight) value[j] *= s.out_weight[s.norm_all ? head * s.vdim + c + j : c + j];
+                if (s.gate_kind) {
+                    const float sig = 1.0f / (1.0f + expf(-g[j]));
+                    value[j] *= s.gate_kind == 2 ? g[j] * sig : sig;
+                }
+                value[j] *= s.out_scale;
+            }
+            store_group<V>(orow + c, value);
         }
     }
     mlr_grid_dependents_may_start();
@@ -1002,6 +1026,19 @@ static int check_recurrence(const RecurrenceSpec& s) {
     return 0;
 }
 
+namespace {
+template <typename T>
+void launch_readout(const RecurrenceSpec& s, const float* obuf, const T* side, int ld_side, const float* gf, T* out, int ld_out, int rows,
+                    cudaStream_t stream) {
+    const auto aligned = [](const void* p, size_t bytes) { return reinterpret_cast<uintptr_t>(p) % bytes == 0; };
+    // Head sizes that are no multiple of 32 keep the one-kernel form's order of every sum (the same bits in both forms).
+    const bool vec = s.dim % 32 == 0 && s.vdim % 4 == 0 && aligned(obuf, 16) && aligned(out, 4 * sizeof(T)) && ld_out % 4 == 0 &&
+                     (!s.gate_kind || (gf ? aligned(gf, 16) : aligned(side + s.col_gate, 4 * sizeof(T)) && ld_side % 4 == 0));
+    if (vec) mlr_launch((recurrence_readout_kernel<T, true>), dim3(rows), dim3(kReadoutThreads), 0, stream, obuf, side, ld_side, gf, out, ld_out, s);
+    else mlr_launch((recurrence_readout_kernel<T, false>), dim3(rows), dim3(kReadoutThreads), 0, stream, obuf, side, ld_side, gf, out, ld_out, s);
+}
+}  // namespace
+
 MLR_API int mlr_linear_recurrence(const RecurrenceSpec* spec, const void* proj, int ld, const void* side, int ld_side, int act_bf16, void* out, int ld_out,
                                   float* state, long long state_stride, const int* segment_info, int n_segments, int rows, float* obuf,
                                   int* status, cudaStream_t stream) {
@@ -1052,12 +1089,8 @@ MLR_API int mlr_linear_recurrence(const RecurrenceSpec* spec, const void* proj, 
 #undef MLR_GO
 #undef MLR_GO2
     if (obuf && rows > 0) {
-        if (act_bf16)
-            mlr_launch((recurrence_readout_kernel<__nv_bfloat16>), dim3(rows), dim3(128), 0, stream, obuf, static_cast<const __nv_bfloat16*>(side),
-                       ld_side, static_cast<const float*>(nullptr), static_cast<__nv_bfloat16*>(out), ld_out, s);
-        else
-            mlr_launch((recurrence_readout_kernel<float>), dim3(rows), dim3(128), 0, stream, obuf, static_cast<const float*>(side), ld_side,
-                       static_cast<const float*>(nullptr), static_cast<float*>(out), ld_out, s);
+        if (act_bf16) launch_readout(s, obuf, static_cast<const __nv_bfloat16*>(side), ld_side, nullptr, static_cast<__nv_bfloat16*>(out), ld_out, rows, stream);
+        else launch_readout(s, obuf, static_cast<const float*>(side), ld_side, nullptr, static_cast<float*>(out), ld_out, rows, stream);
     }
     return mlr_launched("linear_recurrence");
 }
@@ -1129,8 +1162,8 @@ MLR_API int mlr_linear_recurrence_split(const RecurrenceSpec* spec, const void* 
         } else {                                                                                                                       \
             MLR_SCAN(T, false);                                                                                                        \
         }                                                                                                                              \
-        mlr_launch((recurrence_readout_kernel<T>), dim3(rows), dim3(128), 0, stream, obuf, static_cast<const T*>(side), ld_side,       \
-                   static_cast<const float*>(s.gate_rank ? gf : nullptr), static_cast<T*>(out), ld_out, s);                            \
+        launch_readout(s, obuf, static_cast<const T*>(side), ld_side, static_cast<const float*>(s.gate_rank ? gf : nullptr),           \
+                       static_cast<T*>(out), ld_out, rows, stream);                                                                    \
     } while (0)
     if (act_bf16) MLR_SPLIT(__nv_bfloat16);
     else MLR_SPLIT(float);
