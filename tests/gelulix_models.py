@@ -53,7 +53,7 @@ ALL = {
         _delta(4, 2, 32, 64, 4, (8, 24)), _latent(2, 64, 64, 16, 64, 0.1, 300.0, (32.0, 16, 1.0, 0.1))]),
     "only_gla": _model(61, 32, 1e-5, 1.5, [_gla(2, 16, 12, 6.0, 4), _gla(4, 96, 8, 2.0, 8, ff=16)]),
     "only_delta": _model(61, 32, 1e-5, 3.5, [_delta(4, 2, 12, 16, 3, (4, 6), ff=24), _delta(1, 1, 16, 40, 4, (8, 8))]),
-    "only_latent": _model(61, 32, 1e-5, 1.2, [_latent(2, 16, 8, 16, 24, 0.3, 20.0, (3.0, 32, 2.0, 0.5)), _latent(4, 8, 16, 24, 48, 0.2, 1000.0, ff=16)]),
+    "only_latent": _model(61, 32, 1e-5, 1.2, [_latent(2, 16, 8, 16, 24, 0.3, 20.0, (3.0, 32, 2.0, 0.5)), _latent(4, 8, 16, 24, 272, 0.2, 1000.0, ff=16)]),
 }
 
 
