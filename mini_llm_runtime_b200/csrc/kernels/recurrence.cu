@@ -309,10 +309,13 @@ __global__ void __launch_bounds__(1024) linear_recurrence_kernel(const T* proj, 
 // preparation and the read-out are parallel over rows, and the scan, the only sequential part, has a block per
 // (request, head, group of 16 columns of the state).
 
-// q and k of every row, prepared, as float32 [rows, qk_heads * dim] each; for the delta rule also g and beta [rows, 2 * heads].
+// q and k of every row, prepared, as float32 [rows, qk_heads * dim] each; for the delta rule also g and beta [rows, 2 * heads].  zf
+// (or null): [rows, heads * dim], z of every key channel without its bias, turned into the channel's decay in place.
+constexpr int kPrepareThreads = 256;
+
 template <typename T>
-__global__ void __launch_bounds__(128) recurrence_prepare_kernel(const T* proj, int ld, const T* side, int ld_side, float* qf, float* kf,
-                                                                 float* gates, const int* positions, RecurrenceSpec s) {
+__global__ void __launch_bounds__(kPrepareThreads) recurrence_prepare_kernel(const T* proj, int ld, const T* side, int ld_side, float* qf, float* kf,
+                                                                            float* gates, float* zf, const int* positions, RecurrenceSpec s) {
     mlr_grid_wait();
     const int row = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -356,6 +359,20 @@ __global__ void __launch_bounds__(128) recurrence_prepare_kernel(const T* proj, 
             if (!s.channel_decay)
                 gates[static_cast<size_t>(row) * 2 * s.heads + h] = expf(-expf(s.a_log[h]) * softplus(mlr_load(sd, s.col_a + h) + s.dt_bias[h]));
             gates[static_cast<size_t>(row) * 2 * s.heads + s.heads + h] = 1.0f / (1.0f + expf(-b));
+        }
+    }
+    if (zf) {
+        const int channels = s.heads * s.dim;
+        float* z = zf + static_cast<size_t>(row) * channels;
+        if (s.dim % 4 == 0) {                    // four channels of one head an access
+            for (int c = threadIdx.x * 4; c < channels; c += blockDim.x * 4) {
+                const float4 x = __ldcg(reinterpret_cast<const float4*>(z + c)), b = *reinterpret_cast<const float4*>(s.dt_bias + c);
+                const int head = c / s.dim;
+                *reinterpret_cast<float4*>(z + c) = make_float4(channel_decay_of(s, x.x + b.x, head), channel_decay_of(s, x.y + b.y, head),
+                                                                channel_decay_of(s, x.z + b.z, head), channel_decay_of(s, x.w + b.w, head));
+            }
+        } else {
+            for (int c = threadIdx.x; c < channels; c += blockDim.x) z[c] = channel_decay_of(s, __ldcg(z + c) + s.dt_bias[c], c / s.dim);
         }
     }
     mlr_grid_dependents_may_start();
@@ -1097,11 +1114,12 @@ MLR_API int mlr_linear_recurrence(const RecurrenceSpec* spec, const void* proj, 
 
 // The three-kernel form.  qf, kf: float32 [rows, qk_heads * dim]; gates: float32 [rows, 2 * heads] (delta rule; else unused);
 // obuf: float32 [rows, heads * vdim].  Same results as `mlr_linear_recurrence` up to the order in which a column's sums are added
-// (the same order for head sizes that are no multiple of 32).
+// (the same order for head sizes that are no multiple of 32).  With a decay per channel, df [rows, heads * dim] and (low-rank gate) gf
+// [rows, heads * vdim] are float32 room; with `products_made` they hold the low-rank products' results already (df without the bias).
 MLR_API int mlr_linear_recurrence_split(const RecurrenceSpec* spec, const void* proj, int ld, const void* side, int ld_side, int act_bf16,
                                         void* out, int ld_out, float* state, long long state_stride, const int* segment_info,
                                         int n_segments, const int* positions, int rows, float* qf, float* kf, float* gates, float* obuf,
-                                        float* df, float* gf, cudaStream_t stream) {
+                                        float* df, float* gf, int products_made, cudaStream_t stream) {
     MLR_REQUIRE(spec, "linear_recurrence_split: no description");
     const RecurrenceSpec& s = *spec;
     if (check_recurrence(s)) return 1;
@@ -1148,9 +1166,11 @@ MLR_API int mlr_linear_recurrence_split(const RecurrenceSpec* spec, const void* 
     } while (0)
 #define MLR_SPLIT(T)                                                                                                                   \
     do {                                                                                                                               \
-        mlr_launch((recurrence_prepare_kernel<T>), dim3(rows), dim3(128), 0, stream, static_cast<const T*>(proj), ld,                  \
-                   static_cast<const T*>(side), ld_side, qf, kf, gates, positions, s);                                                 \
-        if (channel) {                                                                                                                 \
+        mlr_launch((recurrence_prepare_kernel<T>), dim3(rows), dim3(kPrepareThreads), 0, stream, static_cast<const T*>(proj), ld,      \
+                   static_cast<const T*>(side), ld_side, qf, kf, gates, channel && products_made ? df : nullptr, positions, s);        \
+        if (channel && products_made) {                                                                                                \
+            MLR_SCAN(T, true);                                                                                                         \
+        } else if (channel) {                                                                                                                 \
             if (channel_shared > 48 * 1024)                                                                                            \
                 cudaFuncSetAttribute(group == 4 ? recurrence_channel_kernel<T, 4> : recurrence_channel_kernel<T, 1>,                   \
                                      cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(channel_shared));                   \

@@ -24,7 +24,7 @@ from ..config.registry import register_part
 from ..ops import functions as F
 from ..ops.specs import GATES, RecurrenceSpec, address
 from ..weights.loader import WeightSpec
-from .base import RunContext, SequenceCore, StateNeed
+from .base import RunContext, SequenceCore, StateNeed, columns_of
 from .rotary import plain_rotation
 
 
@@ -41,16 +41,26 @@ def emit_recurrence(b, mixer, proj, side, act, run: RunContext) -> None:
                  act.ptr, act.ld, state.data_ptr(), state.stride(0), info, b.segments, proj.rows, plain.ptr if plain else None,
                  b.status, b.stream)
         return
-    # A decay per key channel, and a gate that comes of a product of small rank, are made for all rows beforehand.
-    df = b.temp(proj.rows, d.heads * d.dim, torch.float32) if d.channel_decay else None
-    gf = b.temp(proj.rows, d.heads * d.vdim, torch.float32) if d.gate_rank else None
+    # A decay per key channel, and a gate that comes of a product of small rank, are made for all rows beforehand: by the matrix
+    # product where its operand (a few columns of the projections) starts on a 16-byte border, else by a kernel of the family.
+    df = gf = None
+    made = 0
+    if d.channel_decay:
+        halves = [(d.col_a, mixer.second_decay)] + ([(d.col_gate, mixer.second_gate)] if d.gate_rank else [])
+        made = int(b.rt.is_bf16 and all(at % 8 == 0 and w.shape[1] % 8 == 0 and w.shape[0] % 8 == 0 for at, w in halves) and side.ld % 8 == 0)
+        if made:
+            df = b.rt.linear(b, columns_of(side, d.col_a, d.decay_rank), mixer.second_decay, out_dtype=torch.float32, activation=True)
+            gf = b.rt.linear(b, columns_of(side, d.col_gate, d.gate_rank), mixer.second_gate, out_dtype=torch.float32, activation=True) if d.gate_rank else None
+        else:
+            df = b.temp(proj.rows, d.heads * d.dim, torch.float32)
+            gf = b.temp(proj.rows, d.heads * d.vdim, torch.float32) if d.gate_rank else None
     qf = b.temp(proj.rows, d.qk_heads * d.dim, torch.float32)
     kf = b.temp(proj.rows, d.qk_heads * d.dim, torch.float32)
     gates = b.temp(proj.rows, 2 * d.heads, torch.float32)
     obuf = b.temp(proj.rows, d.heads * d.vdim, torch.float32)
     b.launch("recurrence", "mlr_linear_recurrence_split", address(d), proj.ptr, proj.ld, side.ptr, side.ld, proj.is_bf16, act.ptr,
              act.ld, state.data_ptr(), state.stride(0), info, b.segments, b.meta("positions"), proj.rows, qf.ptr, kf.ptr, gates.ptr,
-             obuf.ptr, df.ptr if df else None, gf.ptr if gf else None, b.stream)
+             obuf.ptr, df.ptr if df else None, gf.ptr if gf else None, made, b.stream)
 
 
 def _check_state_size(dim: int, vdim: int) -> None:
@@ -266,9 +276,10 @@ def _check_rank(rank: int, what: str) -> int:
     return rank
 
 
-def _second_half(tensors, name: str, rt) -> torch.Tensor:
-    """[rank, outputs]: the second matrix of a low-rank product as the recurrence kernels read it."""
-    return rt.matrix(tensors[name]).t().contiguous()
+def _second_half(tensors, name: str, rt) -> Tuple[torch.Tensor, torch.Tensor]:
+    """The second matrix of a low-rank product: [outputs, rank] for the matrix product, [rank, outputs] as the recurrence kernels read it."""
+    w = rt.matrix(tensors[name]).contiguous()
+    return w, w.t().contiguous()
 
 
 class GatedLinearMixer(SequenceCore):
@@ -316,7 +327,8 @@ class GatedLinearMixer(SequenceCore):
         w = self.spec.weights
         at = self.in_columns()
         vec = lambda role: rt.vector(tensors[w[role]]).float().contiguous()
-        self._held = (vec("a2_bias"), vec("norm"), _second_half(tensors, w["a2"], rt))
+        self.second_decay, turned = _second_half(tensors, w["a2"], rt)
+        self._held = (vec("a2_bias"), vec("norm"), turned)
         self.desc = RecurrenceSpec(
             dt_bias=self._held[0].data_ptr(), out_weight=self._held[1].data_ptr(), decay_w=self._held[2].data_ptr(), heads=self.heads,
             qk_heads=self.heads, dim=self.dim, vdim=self.vdim, prep=RecurrenceSpec.PREP[None], rot_dims=0, rule=RecurrenceSpec.RULE["decay"],
@@ -346,8 +358,8 @@ class ChannelDeltaMixer(DeltaRuleMixer):
         self.gate_rank = _check_rank(int(spec.params["gate_rank"]), "gate")
 
     def in_roles(self) -> List[Tuple[str, int]]:
-        return [("q", self.qk_heads * self.dim), ("k", self.qk_heads * self.dim), ("v", self.heads * self.vdim), ("b", self.heads),
-                ("a1", self.decay_rank), ("g1", self.gate_rank)]
+        return [("q", self.qk_heads * self.dim), ("k", self.qk_heads * self.dim), ("v", self.heads * self.vdim),
+                ("a1", self.decay_rank), ("g1", self.gate_rank), ("b", self.heads)]
 
     def extra_weight_specs(self) -> List[WeightSpec]:
         w = self.spec.weights
@@ -358,7 +370,9 @@ class ChannelDeltaMixer(DeltaRuleMixer):
 
     def _channel_weights(self, tensors, rt) -> tuple:
         w = self.spec.weights
-        self._seconds = (_second_half(tensors, w["a2"], rt), _second_half(tensors, w["g2"], rt))
+        self.second_decay, decay = _second_half(tensors, w["a2"], rt)
+        self.second_gate, gate = _second_half(tensors, w["g2"], rt)
+        self._seconds = (decay, gate)
         return self._seconds
 
     def _describe(self, at) -> None:

@@ -360,7 +360,7 @@ def _recurrence_case(dtype, rule, heads, qk_heads, dim, vdim, rot_dims, segments
             _call("recurrence", "mlr_linear_recurrence_split", ctypes.addressof(spec), proj.data_ptr(), proj.stride(0), proj.data_ptr(),
                   proj.stride(0), native.is_bf16(proj), out.data_ptr(), out.stride(0), state.data_ptr(), state.stride(0),
                   seg_info.data_ptr(), len(segments), positions.data_ptr(), rows, qf.data_ptr(), kf.data_ptr(), gb.data_ptr(),
-                  obuf.data_ptr(), None, None, native.stream())
+                  obuf.data_ptr(), None, None, 0, native.stream())
         else:
             _call("recurrence", "mlr_linear_recurrence", ctypes.addressof(spec), proj.data_ptr(), proj.stride(0), proj.data_ptr(),
                   proj.stride(0), native.is_bf16(proj), out.data_ptr(), out.stride(0), state.data_ptr(), state.stride(0),
