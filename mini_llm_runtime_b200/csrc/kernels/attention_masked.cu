@@ -12,6 +12,8 @@
 //               slopes[head] * (p - j), a bias that grows with the distance
 //   sink:       softmax with exp(sink_h) added to the denominator (a key without a value whose score is a learned number
 //               per head, or 0 where none is given)
+//   maps:       differential attention (`maps` 2 of the description): two softmaxes a head, each with queries and keys of its own, over
+//               the same values; the result is their weighted difference over its root mean square.  A block takes both maps of a head.
 //   gate:       out *= sigmoid(gate) or silu(gate), element by element (or sigmoid of ONE value per head), and a constant factor
 //
 // Cache of a layer: per page, the keys [kv_head][token_in_page][dim] and then the values
@@ -23,28 +25,9 @@
 // the float32 path and sizes the others do not take.  In bfloat16, decoded tokens and short portions go to a kernel whose
 // block holds all query heads of ONE kv head (the heads are the rows of its tensor-core tiles, so a range of keys is read
 // once for the group), and `mlr_attention_masked_tiles` (below) takes the prompt portions in tiles of 64 rows.
+#include "attention_spec.cuh"
 #include "common.cuh"
 #include <type_traits>
-
-struct MaskedAttentionSpec {
-    const float* freq;     // [rot_dims / 2] float32 on the device, or null
-    const float* sinks;    // [heads] float32 on the device: the sink's score per head; null with sink set: 0
-    const float* slopes;   // [heads] float32 on the device: score -= slopes[head] * distance; null: no such bias
-    const float* q_weight; // the weights of a norm of q and of k that `mlr_qkv_prepare_cache` applies (float32 on the device):
-    const float* k_weight; // qk_norm 1: [dim] each, shared by all heads; qk_norm 2: [heads * dim] and [kv_heads * dim]
-    int heads, kv_heads, dim, vdim;
-    int rot_dims, window, chunk, sink;
-    int gate_kind;         // 0 none, 1 sigmoid, 2 silu, 3 sigmoid of one value per head (the gate has `heads` columns)
-    int shared_kv;         // 1: a token's value is the first vdim values of its key (vdim <= dim; one vector per token is cached and a page holds keys only)
-    int keep_first;        // with a window: the first keep_first positions stay visible
-    int qk_norm;           // 0 none; 1 every head of q and k over its root mean square, times a weight; 2 the WHOLE projection (all heads) likewise
-    int dense_cache;       // 1: `mlr_qkv_prepare_cache` serves the kernels of the plain causal attention (attention_bf16, attention_tcgen05,
-                           // attention_generic) instead of this file's: it also rotates the queries in place, and writes the cache as those
-                           // kernels read it ([page][K | V][kv_head][token][dim] with dim = vdim, bfloat16 rows of 64, 128 or 256 values with
-                           // their 16-byte chunks swizzled by the position: `mlr_cache_col`)
-    float scale, out_scale;
-    float softcap;         // > 0: score <- softcap * tanh(score / softcap)
-};
 
 // What a score becomes after the product: scaled, capped, biased by the distance to the key.
 __device__ __forceinline__ float mlr_masked_score(float dot, int distance, float slope, const MaskedAttentionSpec& s) {
@@ -72,6 +55,23 @@ __device__ __forceinline__ int partial_slots(const MaskedAttentionSpec& s) {
     return max(kRowsPerItem * s.kv_heads, ((s.heads + kRowsPerItem - 1) / kRowsPerItem) * kRowsPerItem);
 }
 
+
+// The two maps' results of a head in the registers of a block of kThreads threads (DPT columns each) to the head's result.
+template <typename T, int DPT>
+__device__ __forceinline__ void store_difference(T* orow, const float (&first)[DPT], const float (&second)[DPT], const MaskedAttentionSpec& s, float* scratch) {
+    float value[DPT], squares = 0.0f;
+#pragma unroll
+    for (int d = 0; d < DPT; ++d) {
+        value[d] = threadIdx.x + d * kThreads < s.vdim ? fmaf(-s.map_weight, second[d], first[d]) : 0.0f;
+        squares = fmaf(value[d], value[d], squares);
+    }
+    const float inv = s.out_scale / sqrtf(mlr_block_sum(squares, scratch) / static_cast<float>(s.vdim) + s.map_eps);
+#pragma unroll
+    for (int d = 0; d < DPT; ++d) {
+        const int c = threadIdx.x + d * kThreads;
+        if (c < s.vdim) mlr_store(orow, c, value[d] * inv);
+    }
+}
 
 template <typename T>
 __global__ void __launch_bounds__(kThreads) kv_rope_cache_kernel(const T* k, int ld_k, const T* v, int ld_v, T* cache, int num_pages,
@@ -256,9 +256,13 @@ __global__ void __launch_bounds__(kThreads) attention_masked_kernel(const T* q, 
         first_row = info[0];
         n_rows = min(info[1], kRowsPerItem);
     }
-    const int head = blockIdx.y;
+    const int maps = attention_maps(s), key_row = attention_key_row(s);
+    __shared__ float scratch[32];
     auto one_row = [&](const int row, const int j) {
-    __syncthreads();            // the row before is done with the shared memory
+    float results[2][DPT];      // differential attention: the two maps' results
+    for (int map = 0; map < maps; ++map) {
+    const int head = blockIdx.y * maps + map;
+    __syncthreads();            // the row (or map) before is done with the shared memory
     const int kv_head = head / (s.heads / s.kv_heads);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int position = positions[row];
@@ -270,8 +274,8 @@ __global__ void __launch_bounds__(kThreads) attention_masked_kernel(const T* q, 
     const float slope = s.slopes ? s.slopes[head] : 0.0f;
     const float sink_score = s.sinks ? s.sinks[head] : 0.0f;
     const int* table = block_table + static_cast<size_t>(segment) * table_stride;
-    const size_t page_elems = static_cast<size_t>(s.kv_heads) * page_size * (s.shared_kv ? s.dim : s.dim + s.vdim);
-    const size_t key_plane = s.shared_kv ? 0 : static_cast<size_t>(s.kv_heads) * page_size * s.dim;
+    const size_t page_elems = static_cast<size_t>(s.kv_heads) * page_size * (s.shared_kv ? s.dim : key_row + s.vdim);
+    const size_t key_plane = s.shared_kv ? 0 : static_cast<size_t>(s.kv_heads) * page_size * key_row;
     const int value_row = s.shared_kv ? s.dim : s.vdim;      // values between two tokens' value rows
 
     const T* qrow = q + static_cast<size_t>(row) * ldq + static_cast<size_t>(head) * s.dim;
@@ -303,7 +307,7 @@ __global__ void __launch_bounds__(kThreads) attention_masked_kernel(const T* q, 
     }
 
     constexpr int kChunk = 16 / sizeof(T);                      // values in 16 bytes
-    const bool chunked_rows = s.dim % kChunk == 0;              // a key's row is whole 16-byte pieces, each aligned
+    const bool chunked_rows = s.dim % kChunk == 0;              // a key (of a map) is whole 16-byte pieces, each aligned
     // The kept first keys come first, as tiles of their own (of the first key range only); then the window's tiles.
     const int kept_tiles = (kept > 0 && (!partial || blockIdx.z == 0)) ? (kept + kTile - 1) / kTile : 0;
     const int main_tiles = (tile_last - tile_first) / kTile + 1;
@@ -321,7 +325,7 @@ __global__ void __launch_bounds__(kThreads) attention_masked_kernel(const T* q, 
                 if (page < 0 || page >= num_pages) {
                     bad = 1;
                 } else {
-                    const T* k = cache + page * page_elems + (static_cast<size_t>(kv_head) * page_size + t % page_size) * s.dim;
+                    const T* k = cache + page * page_elems + (static_cast<size_t>(kv_head) * page_size + t % page_size) * key_row + map * s.dim;
                     offset = static_cast<long long>(page * page_elems + key_plane +
                                                     (static_cast<size_t>(kv_head) * page_size + t % page_size) * value_row);
                     for (int c0 = (threadIdx.x & 1) * kChunk; c0 < s.dim; c0 += 8 * kChunk) {     // four pieces on their way at a time
@@ -360,7 +364,7 @@ __global__ void __launch_bounds__(kThreads) attention_masked_kernel(const T* q, 
                 if (page < 0 || page >= num_pages) {
                     if (lane == 0) bad = 1;
                 } else {
-                    const T* k = cache + page * page_elems + (static_cast<size_t>(kv_head) * page_size + t % page_size) * s.dim;
+                    const T* k = cache + page * page_elems + (static_cast<size_t>(kv_head) * page_size + t % page_size) * key_row + map * s.dim;
                     offset = static_cast<long long>(page * page_elems + key_plane +
                                                     (static_cast<size_t>(kv_head) * page_size + t % page_size) * value_row);
                     float partial = 0.0f;
@@ -424,7 +428,15 @@ __global__ void __launch_bounds__(kThreads) attention_masked_kernel(const T* q, 
             const int c = threadIdx.x + d * kThreads;
             if (c < s.vdim) mine[2 + c] = acc[d];
         }
-        return;
+        continue;
+    }
+    if (maps > 1) {
+#pragma unroll
+        for (int d = 0; d < DPT; ++d) {
+            const float value = running_sum > 0.0f ? acc[d] / running_sum : 0.0f;
+            if (map == 0) results[0][d] = value; else results[1][d] = value;
+        }
+        continue;
     }
     T* orow = out + static_cast<size_t>(row) * ldo + static_cast<size_t>(head) * s.vdim;
     const T* grow = gate ? gate + static_cast<size_t>(row) * ld_gate + static_cast<size_t>(head) * (s.gate_kind == 3 ? 1 : s.vdim) : nullptr;
@@ -437,6 +449,9 @@ __global__ void __launch_bounds__(kThreads) attention_masked_kernel(const T* q, 
             mlr_store(orow, c, value * s.out_scale);
         }
     }
+    }
+    if (maps > 1 && !partial)
+        store_difference<T, DPT>(out + static_cast<size_t>(row) * ldo + static_cast<size_t>(blockIdx.y) * s.vdim, results[0], results[1], s, scratch);
     };
     for (int j = 0; j < n_rows; ++j) one_row(first_row + j, j);
     mlr_grid_dependents_may_start();
@@ -448,10 +463,14 @@ __global__ void __launch_bounds__(kThreads) attention_masked_merge_kernel(const 
                                                                           const int* positions, MaskedAttentionSpec s, const int* items,
                                                                           const int* segment_info, int split_keys, int max_splits) {
     mlr_grid_wait();
-    const int item = blockIdx.x, head = blockIdx.y;
+    const int item = blockIdx.x, maps = attention_maps(s);
+    __shared__ float scratch[32];
     const int* info = segment_info + 4 * (items ? items[item] : item);
     for (int j = 0; j < min(info[1], kRowsPerItem); ++j) {
     const int row = info[0] + j;
+    float results[2][DPT];
+    for (int map = 0; map < maps; ++map) {
+    const int head = blockIdx.y * maps + map;
     const int position = positions[row];
     int lo = 0;
     if (s.window > 0) lo = max(lo, position - s.window + 1);
@@ -475,6 +494,14 @@ __global__ void __launch_bounds__(kThreads) attention_masked_merge_kernel(const 
             if (c < s.vdim) acc[d] = fmaf(__ldcg(part + 2 + c), w, acc[d]);
         }
     }
+    if (maps > 1) {
+#pragma unroll
+        for (int d = 0; d < DPT; ++d) {
+            const float value = sum > 0.0f ? acc[d] / sum : 0.0f;
+            if (map == 0) results[0][d] = value; else results[1][d] = value;
+        }
+        continue;
+    }
     T* orow = out + static_cast<size_t>(row) * ldo + static_cast<size_t>(head) * s.vdim;
     const T* grow = gate ? gate + static_cast<size_t>(row) * ld_gate + static_cast<size_t>(head) * (s.gate_kind == 3 ? 1 : s.vdim) : nullptr;
 #pragma unroll
@@ -486,6 +513,9 @@ __global__ void __launch_bounds__(kThreads) attention_masked_merge_kernel(const 
             mlr_store(orow, c, value * s.out_scale);
         }
     }
+    }
+    if (maps > 1)
+        store_difference<T, DPT>(out + static_cast<size_t>(row) * ldo + static_cast<size_t>(blockIdx.y) * s.vdim, results[0], results[1], s, scratch);
     }
     mlr_grid_dependents_may_start();
 }
@@ -543,30 +573,32 @@ __device__ __forceinline__ int first_visible(int position, const MaskedAttention
     return lo;
 }
 
-template <int NV>
-__global__ void __launch_bounds__(128) attention_masked_tile_kernel(const __nv_bfloat16* q, int ldq, const __nv_bfloat16* gate, int ld_gate,
+// MAPS 2 (differential attention): eight warps, four per map; the first map's warps combine both maps' results.
+template <int NV, int MAPS>
+__global__ void __launch_bounds__(128 * MAPS) attention_masked_tile_kernel(const __nv_bfloat16* q, int ldq, const __nv_bfloat16* gate, int ld_gate,
                                                                     __nv_bfloat16* out, int ldo, const __nv_bfloat16* cache, int num_pages,
                                                                     const int* tiles, const int* segment_info, const int* block_table,
                                                                     int table_stride, int page_size, MaskedAttentionSpec s, int* status) {
     mlr_grid_wait();
     extern __shared__ __align__(16) unsigned char smem[];
-    const int qstride = s.dim + kPad, vstride = s.shared_kv ? qstride : s.vdim + kPad;
+    // A row of Q or K holds all maps' values side by side.
+    const int key_row = MAPS * s.dim, qstride = key_row + kPad, vstride = s.shared_kv ? qstride : s.vdim + kPad;
     __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem);
     __nv_bfloat16* Ks = Qs + kRows * qstride;
     __nv_bfloat16* Vs = s.shared_kv ? Ks : Ks + 2 * kKeys * qstride;        // two stages of each; values that are their keys' start are read there
     __shared__ int bad;
 
     const int tile_index = blockIdx.y;       // the planner lists the tiles that see the most keys first
-    const int head = blockIdx.x, kv_head = head / (s.heads / s.kv_heads);
+    const int head = blockIdx.x, kv_head = head * MAPS / (s.heads / s.kv_heads);
     const int segment = tiles[2 * tile_index], tile_token = tiles[2 * tile_index + 1];
     const int first = segment_info[4 * segment], count = segment_info[4 * segment + 1], start = segment_info[4 * segment + 2];
     const int n_rows = min(kRows, count - tile_token);
     const int first_pos = start + tile_token, last_pos = first_pos + n_rows - 1;
     const int lo_min = first_visible(first_pos, s);
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
+    const int lane = threadIdx.x & 31, warp = (threadIdx.x >> 5) & 3, map = threadIdx.x >> 7, g = lane >> 2, t = lane & 3;
     const int* table = block_table + static_cast<size_t>(segment) * table_stride;
-    const size_t page_elems = static_cast<size_t>(s.kv_heads) * page_size * (s.shared_kv ? s.dim : s.dim + s.vdim);
-    const size_t key_plane = s.shared_kv ? 0 : static_cast<size_t>(s.kv_heads) * page_size * s.dim;
+    const size_t page_elems = static_cast<size_t>(s.kv_heads) * page_size * (s.shared_kv ? s.dim : key_row + s.vdim);
+    const size_t key_plane = s.shared_kv ? 0 : static_cast<size_t>(s.kv_heads) * page_size * key_row;
     const int value_row = s.shared_kv ? s.dim : s.vdim;
     const int keep_first = s.window > 0 ? s.keep_first : 0;
     const float slope = s.slopes ? s.slopes[head] : 0.0f;
@@ -578,13 +610,13 @@ __global__ void __launch_bounds__(128) attention_masked_tile_kernel(const __nv_b
 
     // The block's queries, rotated in float32, as bfloat16.
     const int half = s.rot_dims / 2;
-    for (int i = threadIdx.x; i < kRows * s.dim; i += 128) {
-        const int r = i / s.dim, c = i % s.dim;
+    for (int i = threadIdx.x; i < kRows * key_row; i += 128 * MAPS) {
+        const int r = i / key_row, c = i % key_row;
         float value = 0.0f;
         if (r < n_rows) {
-            const __nv_bfloat16* qrow = q + static_cast<size_t>(first + tile_token + r) * ldq + static_cast<size_t>(head) * s.dim;
+            const __nv_bfloat16* qrow = q + static_cast<size_t>(first + tile_token + r) * ldq + static_cast<size_t>(head) * key_row;
             value = __bfloat162float(qrow[c]);
-            if (c < s.rot_dims) {
+            if (MAPS == 1 && c < s.rot_dims) {
                 float sn, cs;
                 sincosf(static_cast<float>(first_pos + r) * s.freq[c < half ? c : c - half], &sn, &cs);
                 const float other = __bfloat162float(qrow[c < half ? c + half : c - half]);
@@ -605,23 +637,25 @@ __global__ void __launch_bounds__(128) attention_masked_tile_kernel(const __nv_b
     for (int nv = 0; nv < NV; ++nv) O[nv][0] = O[nv][1] = O[nv][2] = O[nv][3] = 0.0f;
     const int ksteps = s.dim / 16;
     const uint32_t vs_base = static_cast<uint32_t>(__cvta_generic_to_shared(Vs));
-    const uint32_t qs_base = static_cast<uint32_t>(__cvta_generic_to_shared(Qs));
-    const uint32_t ks_base = static_cast<uint32_t>(__cvta_generic_to_shared(Ks));
+    // Of a row of Q and K a warp reads its map's values.
+    const uint32_t qs_base = static_cast<uint32_t>(__cvta_generic_to_shared(Qs)) + static_cast<uint32_t>(map * s.dim * 2);
+    const uint32_t ks_base = static_cast<uint32_t>(__cvta_generic_to_shared(Ks)) + static_cast<uint32_t>(map * s.dim * 2);
 
     // Keys and values of a tile of 64 positions go from their pages into one of two stages by asynchronous copies, so
     // that the next tile arrives while this one is multiplied; rows no query of the block may see become zeros.
     // The page of this thread's key of the tile at `kt` (0 where no query of the block sees the key).  It is read one tile
     // before the copies that need it are issued, so that no warp waits for the table between two tiles.
+    constexpr int kSharing = 2 * MAPS;          // threads that copy one key and its value
     auto page_for = [&](int kt) {
-        const int position = kt + (threadIdx.x >> 1);
+        const int position = kt + threadIdx.x / kSharing;
         const bool real = position <= last_pos && (position >= lo_min || position < keep_first);
         return real ? __ldg(table + position / page_size) : 0;
     };
     auto fetch = [&](int kt, int into, int page) {
         __nv_bfloat16* kdst = Ks + into * kKeys * qstride;
         __nv_bfloat16* vdst = Vs + into * kKeys * vstride;
-        // Two threads per key: the row's addresses once, then every other 16-byte piece of the key's row and of its value row.
-        const int key = threadIdx.x >> 1, position = kt + key;
+        // Two threads per key (and map): the row's addresses once, then every other 16-byte piece of the key's row and of its value row.
+        const int key = threadIdx.x / kSharing, position = kt + key, piece = threadIdx.x % kSharing * 8;
         bool real = position <= last_pos && (position >= lo_min || position < keep_first);
         const __nv_bfloat16* ksrc = cache;
         const __nv_bfloat16* vsrc = cache;
@@ -631,15 +665,15 @@ __global__ void __launch_bounds__(128) attention_masked_tile_kernel(const __nv_b
                 real = false;
             } else {
                 const size_t in_page = static_cast<size_t>(kv_head) * page_size + position % page_size;
-                ksrc = cache + page * page_elems + in_page * s.dim;
+                ksrc = cache + page * page_elems + in_page * key_row;
                 vsrc = cache + page * page_elems + key_plane + in_page * value_row;
             }
         }
         __nv_bfloat16* krow = kdst + key * qstride;
         __nv_bfloat16* vrow = vdst + key * vstride;
-        for (int c = (threadIdx.x & 1) * 8; c < s.dim; c += 16) mlr_async_copy16(krow + c, real ? ksrc + c : cache, real);
+        for (int c = piece; c < key_row; c += 8 * kSharing) mlr_async_copy16(krow + c, real ? ksrc + c : cache, real);
         if (!s.shared_kv)
-            for (int c = (threadIdx.x & 1) * 8; c < s.vdim; c += 16) mlr_async_copy16(vrow + c, real ? vsrc + c : cache, real);
+            for (int c = piece; c < s.vdim; c += 8 * kSharing) mlr_async_copy16(vrow + c, real ? vsrc + c : cache, real);
         mlr_async_commit();
     };
     // Tiles of keys in the order they are walked: those of the kept first tokens that lie before the window's first tile, then
@@ -785,6 +819,48 @@ __global__ void __launch_bounds__(128) attention_masked_tile_kernel(const __nv_b
     l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
+    if constexpr (MAPS == 2) {
+        // The second map's results go through shared memory (the values' room) to the warps of the first, which finish the rows.
+        const float inv_a = l_a > 0.0f ? 1.0f / l_a : 0.0f, inv_b = l_b > 0.0f ? 1.0f / l_b : 0.0f;
+        float2* theirs = reinterpret_cast<float2*>(Vs) + (warp * 32 + lane) * 2;         // [piece of 8 columns][warp][lane][upper, lower row]
+        __syncthreads();
+        if (map == 1) {
+#pragma unroll
+            for (int nv = 0; nv < NV; ++nv)
+                if (nv * 8 < s.vdim) {
+                    theirs[nv * 256] = make_float2(O[nv][0] * inv_a, O[nv][1] * inv_a);
+                    theirs[nv * 256 + 1] = make_float2(O[nv][2] * inv_b, O[nv][3] * inv_b);
+                }
+        }
+        __syncthreads();
+        if (map == 1) return;
+        float squares_a = 0.0f, squares_b = 0.0f;
+#pragma unroll
+        for (int nv = 0; nv < NV; ++nv)
+            if (nv * 8 < s.vdim) {
+                const float2 a = theirs[nv * 256], b = theirs[nv * 256 + 1];
+                O[nv][0] = fmaf(-s.map_weight, a.x, O[nv][0] * inv_a);
+                O[nv][1] = fmaf(-s.map_weight, a.y, O[nv][1] * inv_a);
+                O[nv][2] = fmaf(-s.map_weight, b.x, O[nv][2] * inv_b);
+                O[nv][3] = fmaf(-s.map_weight, b.y, O[nv][3] * inv_b);
+                squares_a = fmaf(O[nv][0], O[nv][0], fmaf(O[nv][1], O[nv][1], squares_a));
+                squares_b = fmaf(O[nv][2], O[nv][2], fmaf(O[nv][3], O[nv][3], squares_b));
+            }
+#pragma unroll
+        for (int o = 1; o < 4; o *= 2) {
+            squares_a += __shfl_xor_sync(0xffffffffu, squares_a, o);
+            squares_b += __shfl_xor_sync(0xffffffffu, squares_b, o);
+        }
+        const float scale_a = s.out_scale / sqrtf(squares_a / static_cast<float>(s.vdim) + s.map_eps);
+        const float scale_b = s.out_scale / sqrtf(squares_b / static_cast<float>(s.vdim) + s.map_eps);
+#pragma unroll
+        for (int nv = 0; nv < NV; ++nv) {
+            if (nv * 8 >= s.vdim) continue;
+            __nv_bfloat16* o = out + static_cast<size_t>(first + tile_token + r0 + g) * ldo + head * s.vdim + nv * 8 + 2 * t;
+            if (row_a) *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(O[nv][0] * scale_a, O[nv][1] * scale_a);
+            if (row_b) *reinterpret_cast<__nv_bfloat162*>(o + static_cast<size_t>(8) * ldo) = __floats2bfloat162_rn(O[nv][2] * scale_b, O[nv][3] * scale_b);
+        }
+    } else {
 #pragma unroll
     for (int nv = 0; nv < NV; ++nv) {
         if (nv * 8 >= s.vdim) continue;
@@ -806,6 +882,7 @@ __global__ void __launch_bounds__(128) attention_masked_tile_kernel(const __nv_b
             *reinterpret_cast<__nv_bfloat162*>(out + row * ldo + col) = __floats2bfloat162_rn(v0 * s.out_scale, v1 * s.out_scale);
         }
     }
+    }
 }
 
 // ---- few rows per request in bfloat16 (decoded tokens, short portions): one block per (segment, kv head, range of keys) takes
@@ -824,12 +901,15 @@ __global__ void __launch_bounds__(128, NV >= 16 ? 3 : 4) attention_masked_group_
                                                                      int* status) {
     mlr_grid_wait();
     extern __shared__ __align__(16) unsigned char smem[];
-    const int qstride = s.dim + kPad, vstride = s.shared_kv ? qstride : s.vdim + kPad;
+    // A row of Q or K holds all maps' values side by side; a query has zeros in place of the maps it does not belong to.
+    const int maps = attention_maps(s), key_row = attention_key_row(s);
+    const int qstride = key_row + kPad, vstride = s.shared_kv ? qstride : s.vdim + kPad;
     __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem);
     __nv_bfloat16* Ks = Qs + 16 * qstride;
     __nv_bfloat16* Vs = s.shared_kv ? Ks : Ks + 2 * kKeys * qstride;        // two stages of each; values that are their keys' start are read there
     float* merged = reinterpret_cast<float*>(Ks);                            // [4 warps][16 rows][vdim + 2], once the last tile is done
     __shared__ int bad;
+    __shared__ float scratch[32];
 
     const int* info = segment_info + 4 * (items ? items[blockIdx.x] : blockIdx.x);
     const int first_row = info[0], n_rows = min(info[1], kRowsPerItem);
@@ -838,13 +918,13 @@ __global__ void __launch_bounds__(128, NV >= 16 ? 3 : 4) attention_masked_group_
     const int kv_head = blockIdx.y / chunks, chunk = blockIdx.y % chunks;
     const int head0 = kv_head * sharing + chunk * 16, group = min(16, sharing - chunk * 16);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
-    const size_t page_elems = static_cast<size_t>(s.kv_heads) * page_size * (s.shared_kv ? s.dim : s.dim + s.vdim);
-    const size_t key_plane = s.shared_kv ? 0 : static_cast<size_t>(s.kv_heads) * page_size * s.dim;
+    const size_t page_elems = static_cast<size_t>(s.kv_heads) * page_size * (s.shared_kv ? s.dim : key_row + s.vdim);
+    const size_t key_plane = s.shared_kv ? 0 : static_cast<size_t>(s.kv_heads) * page_size * key_row;
     const bool capped = s.softcap > 0.0f;
     const float to_cap = capped ? 2.0f * 1.4426950408889634f * s.scale / s.softcap : s.scale;
     const float slope_a = (s.slopes && g < group) ? s.slopes[head0 + g] : 0.0f;
     const float slope_b = (s.slopes && g + 8 < group) ? s.slopes[head0 + g + 8] : 0.0f;
-    const int ksteps = s.dim / 16, half = s.rot_dims / 2, mstride = s.vdim + 2;
+    const int ksteps = key_row / 16, half = s.rot_dims / 2, mstride = s.vdim + 2;
     const uint32_t qs_base = static_cast<uint32_t>(__cvta_generic_to_shared(Qs));
     const uint32_t ks_base = static_cast<uint32_t>(__cvta_generic_to_shared(Ks));
     const uint32_t vs_base = static_cast<uint32_t>(__cvta_generic_to_shared(Vs));
@@ -886,12 +966,12 @@ __global__ void __launch_bounds__(128, NV >= 16 ? 3 : 4) attention_masked_group_
                     real = false;
                 } else {
                     const size_t in_page = static_cast<size_t>(kv_head) * page_size + at % page_size;
-                    ksrc = cache + page * page_elems + in_page * s.dim;
+                    ksrc = cache + page * page_elems + in_page * key_row;
                     vsrc = cache + page * page_elems + key_plane + in_page * s.vdim;
                 }
             }
             __nv_bfloat16* krow = Ks + (into * kKeys + key) * qstride;
-            for (int c = (threadIdx.x & 1) * 8; c < s.dim; c += 16) mlr_async_copy16(krow + c, real ? ksrc + c : cache, real);
+            for (int c = (threadIdx.x & 1) * 8; c < key_row; c += 16) mlr_async_copy16(krow + c, real ? ksrc + c : cache, real);
             if (!s.shared_kv) {
                 __nv_bfloat16* vrow = Vs + (into * kKeys + key) * vstride;
                 for (int c = (threadIdx.x & 1) * 8; c < s.vdim; c += 16) mlr_async_copy16(vrow + c, real ? vsrc + c : cache, real);
@@ -902,10 +982,10 @@ __global__ void __launch_bounds__(128, NV >= 16 ? 3 : 4) attention_masked_group_
         fetch(0, 0, page_for(0));
         int page_ahead = all_tiles > 1 ? page_for(1) : 0;
         // The group's queries, rotated in float32, as bfloat16.
-        for (int i = threadIdx.x; i < 16 * s.dim; i += 128) {
-            const int r = i / s.dim, c = i % s.dim;
+        for (int i = threadIdx.x; i < 16 * key_row; i += 128) {
+            const int r = i / key_row, at = i % key_row, c = maps == 1 ? at : at % s.dim;
             float value = 0.0f;
-            if (r < group) {
+            if (r < group && (maps == 1 || at / s.dim == (head0 + r) % maps)) {
                 const __nv_bfloat16* qrow = q + static_cast<size_t>(row) * ldq + static_cast<size_t>(head0 + r) * s.dim;
                 value = __bfloat162float(qrow[c]);
                 if (c < s.rot_dims) {
@@ -915,7 +995,7 @@ __global__ void __launch_bounds__(128, NV >= 16 ? 3 : 4) attention_masked_group_
                     value = c < half ? value * cs - other * sn : value * cs + other * sn;
                 }
             }
-            Qs[r * qstride + c] = __float2bfloat16_rn(value);
+            Qs[r * qstride + at] = __float2bfloat16_rn(value);
         }
         float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.0f, l_b = 0.0f;
         float O[NV][4];
@@ -1042,6 +1122,7 @@ __global__ void __launch_bounds__(128, NV >= 16 ? 3 : 4) attention_masked_group_
             }
         }
         __syncthreads();
+        float before = 0.0f;      // differential attention: the result of the map before (a column a thread; vdim <= 128)
         for (int r = 0; r < group; ++r) {
             const int head = head0 + r;
             float top = -INFINITY, w[4], sum = 0.0f;
@@ -1067,6 +1148,20 @@ __global__ void __launch_bounds__(128, NV >= 16 ? 3 : 4) attention_masked_group_
                     mine[2 + c] = acc;
                 }
             } else {
+                if (maps > 1) {
+                    float value = 0.0f;
+                    if (threadIdx.x < s.vdim) {
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) value = fmaf(merged[(i * 16 + r) * mstride + 2 + threadIdx.x], w[i], value);
+                        value = sum > 0.0f ? value / sum : 0.0f;
+                    }
+                    if (head % maps == 0) before = value;
+                    else {
+                        const float first[1] = {before}, second[1] = {value};
+                        store_difference<__nv_bfloat16, 1>(out + static_cast<size_t>(row) * ldo + static_cast<size_t>(head / maps) * s.vdim, first, second, s, scratch);
+                    }
+                    continue;
+                }
                 // The block saw every key of the row: the sink joins here, and the row is finished.
                 float scale_all = 1.0f;
                 if (s.sink) {
@@ -1105,6 +1200,10 @@ int check_spec(const MaskedAttentionSpec* s, const char* who) {
     MLR_REQUIRE(!s->shared_kv || s->vdim <= s->dim, "%s: values that are the start of their keys cannot be longer, %d against %d", who, s->vdim, s->dim);
     MLR_REQUIRE(s->keep_first >= 0 && (s->keep_first == 0 || (s->window > 0 && s->chunk == 0)), "%s: kept first tokens go with a window and without chunks", who);
     MLR_REQUIRE(s->gate_kind >= 0 && s->gate_kind <= 3 && (!s->sinks || s->sink), "%s: bad gate kind, or sink scores without a sink", who);
+    MLR_REQUIRE(s->maps >= 0 && s->maps <= 2, "%s: one or two attention maps a head, not %d", who, s->maps);
+    MLR_REQUIRE(s->maps < 2 || (s->heads / s->kv_heads % 2 == 0 && s->rot_dims == 0 && !s->sink && !s->slopes && s->gate_kind == 0 && s->softcap <= 0.0f &&
+                                s->keep_first == 0 && !s->shared_kv && !s->dense_cache && s->qk_norm == 0 && s->map_eps >= 0.0f),
+                "%s: two maps a head go with queries that are rotated already, without sink, slopes, gate, cap, kept tokens or values in the keys", who);
     MLR_REQUIRE(!s->dense_cache || (s->dim == s->vdim && !s->shared_kv), "%s: the plain attention kernels' cache has keys and values of one size", who);
     return 0;
 }
@@ -1215,19 +1314,20 @@ MLR_API int mlr_attention_masked(const MaskedAttentionSpec* spec, const void* q,
         }
     }
     MLR_REQUIRE(rows >= 0 && page_size > 0 && num_pages > 0, "attention_masked: bad page size or page count");
-    MLR_REQUIRE(ldq >= spec->heads * spec->dim && ldo >= spec->heads * spec->vdim, "attention_masked: a row stride is smaller than the row");
+    const int maps = attention_maps(*spec), key_row = attention_key_row(*spec);
+    MLR_REQUIRE(ldq >= spec->heads * spec->dim && ldo >= spec->heads / maps * spec->vdim, "attention_masked: a row stride is smaller than the row");
     MLR_REQUIRE((spec->gate_kind == 0) == (gate == nullptr), "attention_masked: the description and the call disagree about a gate");
     if (rows == 0) return 0;
     const size_t shared = sizeof(float) * (spec->dim + kTile) + sizeof(long long) * kTile + 16;
-    const dim3 grid(rows, spec->heads, max_splits);
-    const dim3 merge_grid(rows, spec->heads);
+    const dim3 grid(rows, spec->heads / maps, max_splits);
+    const dim3 merge_grid(rows, spec->heads / maps);
     const int group = spec->heads / spec->kv_heads;
-    if (act_bf16 && segment_info && spec->dim % 16 == 0 && spec->dim <= 256 && spec->vdim % 8 == 0 && spec->vdim <= 128 &&
+    if (act_bf16 && segment_info && spec->dim % 16 == 0 && key_row <= 256 && spec->vdim % 8 == 0 && spec->vdim <= 128 &&
         reinterpret_cast<uintptr_t>(cache) % 16 == 0) {
         // Few rows per request in bfloat16: the query heads of a kv head share one block (and one reading of the keys).
-        const size_t stages = sizeof(__nv_bfloat16) * (static_cast<size_t>(16 + 2 * kKeys) * (spec->dim + kPad) +
+        const size_t stages = sizeof(__nv_bfloat16) * (static_cast<size_t>(16 + 2 * kKeys) * (key_row + kPad) +
                                                        (spec->shared_kv ? 0 : 2 * kKeys * (spec->vdim + kPad)));
-        const size_t sums = sizeof(__nv_bfloat16) * 16 * (spec->dim + kPad) + sizeof(float) * 4 * 16 * (spec->vdim + 2);
+        const size_t sums = sizeof(__nv_bfloat16) * 16 * (key_row + kPad) + sizeof(float) * 4 * 16 * (spec->vdim + 2);
         const size_t group_shared = stages > sums ? stages : sums;
         const dim3 group_grid(rows, spec->kv_heads * ((group + 15) / 16), max_splits);     // more than 16 heads on a kv head: 16 a block
 #define MLR_GROUP(NV)                                                                                                                       \
@@ -1273,7 +1373,7 @@ MLR_API int mlr_attention_masked(const MaskedAttentionSpec* spec, const void* q,
     return mlr_launched("attention_masked");
 }
 
-// Whether the tiled kernel takes these sizes (bfloat16 only): 1 yes, 0 no.
+// Whether the tiled kernel takes these sizes (bfloat16 only; dim: of a key's row, the maps' values side by side): 1 yes, 0 no.
 MLR_API int mlr_attention_masked_tiles_fit(int dim, int vdim) {
     return dim % 16 == 0 && dim >= 16 && dim <= 256 && vdim % 8 == 0 && vdim >= 8 && vdim <= 128;
 }
@@ -1284,21 +1384,27 @@ MLR_API int mlr_attention_masked_tiles(const MaskedAttentionSpec* spec, const vo
                                        const int* segment_info, const int* block_table, int table_stride, int page_size, int* status,
                                        cudaStream_t stream) {
     if (check_spec(spec, "attention_masked_tiles")) return 1;
-    MLR_REQUIRE(mlr_attention_masked_tiles_fit(spec->dim, spec->vdim), "attention_masked_tiles: key size %d / value size %d not taken",
+    const int maps = attention_maps(*spec), key_row = attention_key_row(*spec), out_row = spec->heads / maps * spec->vdim;
+    MLR_REQUIRE(spec->dim % 16 == 0 && mlr_attention_masked_tiles_fit(key_row, spec->vdim), "attention_masked_tiles: key size %d / value size %d not taken",
                 spec->dim, spec->vdim);
     MLR_REQUIRE(n_tiles >= 0 && n_tiles <= 65535 && page_size > 0 && num_pages > 0, "attention_masked_tiles: bad tile count or pages");
-    MLR_REQUIRE(ldq >= spec->heads * spec->dim && ldo >= spec->heads * spec->vdim && ldo % 2 == 0 && (spec->heads * spec->vdim) % 2 == 0,
+    MLR_REQUIRE(ldq >= spec->heads * spec->dim && ldo >= out_row && ldo % 2 == 0 && out_row % 2 == 0,
                 "attention_masked_tiles: bad row strides");
     MLR_REQUIRE((spec->gate_kind == 0) == (gate == nullptr), "attention_masked_tiles: the description and the call disagree about a gate");
     MLR_REQUIRE(reinterpret_cast<uintptr_t>(cache) % 16 == 0 && reinterpret_cast<uintptr_t>(out) % 4 == 0, "attention_masked_tiles: alignment");
     if (n_tiles == 0) return 0;
-    const size_t shared = sizeof(__nv_bfloat16) * (static_cast<size_t>(kRows + 2 * kKeys) * (spec->dim + kPad) +
+    const size_t shared = sizeof(__nv_bfloat16) * (static_cast<size_t>(kRows + 2 * kKeys) * (key_row + kPad) +
                                                    (spec->shared_kv ? 0 : 2 * kKeys * (spec->vdim + kPad)));
-    const dim3 grid(spec->heads, n_tiles);
+    const dim3 grid(spec->heads / maps, n_tiles);
 #define MLR_TILES(NV)                                                                                                              \
     do {                                                                                                                           \
-        cudaFuncSetAttribute(attention_masked_tile_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared)); \
-        mlr_launch((attention_masked_tile_kernel<NV>), dim3(grid), dim3(128), shared, stream, static_cast<const __nv_bfloat16*>(q), ldq, \
+        if (maps == 2) MLR_TILES2(NV, 2);                                                                                          \
+        else MLR_TILES2(NV, 1);                                                                                                    \
+    } while (0)
+#define MLR_TILES2(NV, MAPS)                                                                                                       \
+    do {                                                                                                                           \
+        cudaFuncSetAttribute(attention_masked_tile_kernel<NV, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared)); \
+        mlr_launch((attention_masked_tile_kernel<NV, MAPS>), dim3(grid), dim3(128 * MAPS), shared, stream, static_cast<const __nv_bfloat16*>(q), ldq, \
                    static_cast<const __nv_bfloat16*>(gate), ld_gate, static_cast<__nv_bfloat16*>(out), ldo,                         \
                    static_cast<const __nv_bfloat16*>(cache), num_pages, tiles, segment_info, block_table, table_stride, page_size, \
                    *spec, status);                                                                                                 \
@@ -1308,5 +1414,6 @@ MLR_API int mlr_attention_masked_tiles(const MaskedAttentionSpec* spec, const vo
     else if (spec->vdim <= 96) MLR_TILES(12);
     else MLR_TILES(16);
 #undef MLR_TILES
+#undef MLR_TILES2
     return mlr_launched("attention_masked_tiles");
 }

@@ -211,6 +211,44 @@ __device__ __forceinline__ void mlr_store8(__nv_bfloat16* p, const float (&v)[8]
     *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
 }
 
+// ---- V neighbouring values as float32, through L2 (V = 1: any address; 4: an address aligned to the group) ----
+template <int V, typename T>
+__device__ __forceinline__ void mlr_load_group(const T* p, float* v) {
+    if constexpr (V == 1) {
+        v[0] = mlr_load(p, 0);
+    } else if constexpr (sizeof(T) == 4) {
+#pragma unroll
+        for (int i = 0; i < V; i += 4) {
+            const float4 x = __ldcg(reinterpret_cast<const float4*>(p + i));
+            v[i] = x.x; v[i + 1] = x.y; v[i + 2] = x.z; v[i + 3] = x.w;
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < V; i += 4) {
+            const uint2 x = __ldcg(reinterpret_cast<const uint2*>(p + i));
+            const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&x.x), hi = *reinterpret_cast<const __nv_bfloat162*>(&x.y);
+            const float2 f = __bfloat1622float2(lo), g = __bfloat1622float2(hi);
+            v[i] = f.x; v[i + 1] = f.y; v[i + 2] = g.x; v[i + 3] = g.y;
+        }
+    }
+}
+
+template <int V, typename T>
+__device__ __forceinline__ void mlr_store_group(T* p, const float* v) {
+    if constexpr (V == 1) {
+        mlr_store(p, 0, v[0]);
+    } else if constexpr (sizeof(T) == 4) {
+#pragma unroll
+        for (int i = 0; i < V; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+    } else {
+#pragma unroll
+        for (int i = 0; i < V; i += 4) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(v[i], v[i + 1]), hi = __floats2bfloat162_rn(v[i + 2], v[i + 3]);
+            *reinterpret_cast<uint2*>(p + i) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        }
+    }
+}
+
 // ---- asynchronous copies global -> shared (fire and forget; a thread waits for its own with mlr_async_wait) ----
 __device__ __forceinline__ void mlr_async_copy16(void* shared_dst, const void* global_src, bool real = true) {
     const unsigned dst = static_cast<unsigned>(__cvta_generic_to_shared(shared_dst));

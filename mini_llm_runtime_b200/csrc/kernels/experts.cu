@@ -16,9 +16,15 @@
 //   combine   out[token] = sum_j weight_j y[row of (token, j)]  (+ shared gate * shared expert's result), j in
 //             the order of the choice.
 // A second kind of router (`kind` 1): z = R x + bias (the `correction` operand), the `top` largest z are chosen (ties to
-// the lower index) and their weights are the softmax over the chosen z alone; no groups.  A second shape of the gate
+// the lower index) and their weights are the softmax over the chosen z alone; no groups.  A third (`kind` 2): s = softmax of z over
+// all experts, choice = s + correction, a group's score is its largest choice, and the weights are the chosen s as they are.
+// The last experts of a router may be identity experts (`routed` = how many before them are real): a token that chooses one adds its
+// weight to `identity` [token] and takes no row of the products.  A second shape of the gate
 // (`gated` 2): g <- min(g, limit), u <- clamp(u, -limit, limit) where limit > 0, then g * sigmoid(alpha g) * (u + up_offset).
 #include "common.cuh"
+#include "pieces.cuh"
+
+#include <climits>
 
 namespace {
 
@@ -45,15 +51,34 @@ __device__ __forceinline__ float expert_gate(float g, float u, const ExpertGate&
     return g / (1.0f + expf(-g)) * u;
 }
 
+// The index of the largest value that is no NaN, the lowest of equals; 0 where all are NaN.  All lanes of a warp call it and get it.
+__device__ __forceinline__ int warp_argmax(const float* values, int n) {
+    const int lane = threadIdx.x & 31;
+    float best = -INFINITY;
+    int at = INT_MAX;
+    for (int i = lane; i < n; i += 32) {
+        const float v = values[i];
+        if (!isnan(v) && (at == INT_MAX || v > best)) { best = v; at = i; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float v = __shfl_xor_sync(0xffffffffu, best, o);
+        const int i = __shfl_xor_sync(0xffffffffu, at, o);
+        if (i != INT_MAX && (at == INT_MAX || v > best || (v == best && i < at))) { best = v; at = i; }
+    }
+    return at == INT_MAX ? 0 : at;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kRouteThreads) route_kernel(const T* x, long long ld, const float* router, const float* correction,
-                                                              int width, int experts, int groups, int keep, int top, int has_gate,
-                                                              int* chosen, float* weights, int* place, int* counts, float* shared_gate, int kind) {
+                                                              int width, int experts, int routed, int groups, int keep, int top, int has_gate,
+                                                              int* chosen, float* weights, int* place, int* counts, float* shared_gate,
+                                                              float* identity, int kind) {
     mlr_grid_wait();
     extern __shared__ __align__(16) float shared[];
     float* xs = shared;                 // [width]
     float* score = xs + width;          // [experts] plain scores
-    float* choice = score + experts;    // [experts] scores with the correction (minus infinity once taken or not allowed)
+    float* choice = score + experts;    // [experts] scores with the correction (minus infinity where not allowed, NaN once taken)
     float* group_score = choice + experts;   // [groups]
     const int row = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -79,77 +104,85 @@ __global__ void __launch_bounds__(kRouteThreads) route_kernel(const T* x, long l
         }
         sum = mlr_warp_sum(sum);
         if (lane == 0) {
-            const float s = 1.0f / (1.0f + expf(-sum));
             if (e >= experts) {
-                shared_gate[row] = s;
+                shared_gate[row] = 1.0f / (1.0f + expf(-sum));
+            } else if (kind == 2) {
+                score[e] = sum;
             } else if (kind == 1) {
                 score[e] = choice[e] = sum + (correction ? correction[e] : 0.0f);
             } else {
+                const float s = 1.0f / (1.0f + expf(-sum));
                 score[e] = s;
                 choice[e] = s + (correction ? correction[e] : 0.0f);
             }
         }
     }
     __syncthreads();
-    __shared__ int taken[kMaxTop];
-    __shared__ float picked[kMaxTop];
-    __shared__ float total_score;
-    if (threadIdx.x == 0) {
-    const float none = -INFINITY;
+    if (warp != 0) return;
+    // One warp chooses.
+    if (kind == 2) {
+        float largest = -INFINITY, total = 0.0f;
+        for (int e = lane; e < experts; e += 32) largest = fmaxf(largest, score[e]);
+        largest = mlr_warp_max(largest);
+        for (int e = lane; e < experts; e += 32) {
+            score[e] = expf(score[e] - largest);
+            total += score[e];
+        }
+        total = mlr_warp_sum(total);
+        for (int e = lane; e < experts; e += 32) {
+            score[e] /= total;
+            choice[e] = score[e] + (correction ? correction[e] : 0.0f);
+        }
+        __syncwarp();
+    }
     const int per = experts / groups;
     if (groups > 1 && keep < groups) {
-        for (int g = 0; g < groups; ++g) {
-            float a = none, b = none;           // the two largest of the group
+        for (int g = lane; g < groups; g += 32) {
+            float a = -INFINITY, b = -INFINITY;           // the two largest of the group
             for (int e = g * per; e < (g + 1) * per; ++e) {
                 const float v = choice[e];
                 if (v > a) { b = a; a = v; }
                 else if (v > b) b = v;
             }
-            group_score[g] = per > 1 ? a + b : a;
+            group_score[g] = kind == 0 && per > 1 ? a + b : a;
         }
-        // Groups outside the `keep` best lose their experts: mark the kept ones by taking them out of group_score.
+        __syncwarp();
+        // Groups outside the `keep` best lose their experts; NaN marks a kept one.
         for (int k = 0; k < keep; ++k) {
-            int best = -1;
-            float value = none;
-            for (int g = 0; g < groups; ++g)
-                if (!isnan(group_score[g]) && (best < 0 || group_score[g] > value)) { best = g; value = group_score[g]; }
-            group_score[best] = NAN;            // NaN marks a kept group
+            const int best = warp_argmax(group_score, groups);
+            if (lane == 0) group_score[best] = NAN;
+            __syncwarp();
         }
-        for (int g = 0; g < groups; ++g)
-            if (!isnan(group_score[g]))
-                for (int e = g * per; e < (g + 1) * per; ++e) choice[e] = none;
+        for (int e = lane; e < experts; e += 32)
+            if (!isnan(group_score[e / per])) choice[e] = -INFINITY;
+        __syncwarp();
     }
-    float total = 0.0f;
+    // Lane k holds the k-th chosen expert and its score.
+    int mine = 0;
+    float picked = 0.0f, total = 0.0f, passed = 0.0f;
     for (int k = 0; k < top; ++k) {
-        int best = 0;
-        float value = none;
-        bool found = false;
-        for (int e = 0; e < experts; ++e)
-            if (!isnan(choice[e]) && (!found || choice[e] > value)) { best = e; value = choice[e]; found = true; }
-        choice[best] = NAN;                     // NaN marks a taken expert
-        taken[k] = best;
-        picked[k] = score[best];
-        total += score[best];
+        const int best = warp_argmax(choice, experts);
+        const float s = score[best];
+        if (lane == 0) choice[best] = NAN;                     // NaN marks a taken expert
+        __syncwarp();
+        if (lane == k) { mine = best; picked = s; }
+        total += s;
+        if (best >= routed) passed += s;
     }
     if (kind == 1) {
         // softmax over the chosen logits alone; the first chosen is the largest
-        const float largest = picked[0];
+        picked = expf(picked - __shfl_sync(0xffffffffu, picked, 0));
         total = 0.0f;
-        for (int k = 0; k < top; ++k) {
-            picked[k] = expf(picked[k] - largest);
-            total += picked[k];
-        }
+        for (int k = 0; k < top; ++k) total += __shfl_sync(0xffffffffu, picked, k);
     }
-    total_score = total;
+    // One lane per chosen expert: the counters' answers come back side by side.
+    if (lane < top) {
+        const size_t at = static_cast<size_t>(row) * top + lane;
+        chosen[at] = mine;
+        weights[at] = kind == 2 ? picked : picked / (total + 1e-20f);
+        place[at] = mine < routed ? atomicAdd(counts + mine, 1) : 0;
     }
-    __syncthreads();
-    // One thread per chosen expert: the counters' answers come back side by side.
-    if (threadIdx.x < top) {
-        const int k = threadIdx.x;
-        chosen[static_cast<size_t>(row) * top + k] = taken[k];
-        weights[static_cast<size_t>(row) * top + k] = picked[k] / (total_score + 1e-20f);
-        place[static_cast<size_t>(row) * top + k] = atomicAdd(counts + taken[k], 1);
-    }
+    if (identity && lane == 0) identity[row] = kind == 2 ? passed : passed / (total + 1e-20f);
 }
 
 // One block.  first_row [experts + 1]; tiles: {expert, first row, rows} per tile, n_tiles[0] their number; row_of_pair [pairs]
@@ -183,9 +216,10 @@ __global__ void __launch_bounds__(1024) arrange_kernel(int* counts, const int* c
         counts[e] = 0;
     }
     for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
-        const int row = first[chosen[p]] + place[p];
+        const int expert = chosen[p];
+        const int row = expert < experts ? first[expert] + place[p] : -1;        // an identity expert has no rows
         row_of_pair[p] = row;
-        pair_of_row[row] = p;
+        if (row >= 0) pair_of_row[row] = p;
     }
 }
 
@@ -412,40 +446,34 @@ __global__ void __launch_bounds__(256) expert_product_mma_kernel(const __nv_bflo
         }
 }
 
-template <typename T>
-__global__ void __launch_bounds__(256) combine_kernel(const float* y, long long ldy, const int* row_of_pair, const float* weights, int top,
-                                                      const T* shared_y, long long ld_shared, const float* shared_gate, float* out,
-                                                      long long ldo, int width) {
+template <bool VEC>
+__global__ void __launch_bounds__(256) combine_kernel(Pieces pieces, float* out, long long ldo, int width) {
     mlr_grid_wait();
     const int row = blockIdx.x;
-    __shared__ float weight[kMaxTop];
-    __shared__ long long from[kMaxTop];
-    if (threadIdx.x < top) {
-        weight[threadIdx.x] = __ldcg(weights + row * top + threadIdx.x);
-        from[threadIdx.x] = static_cast<long long>(__ldcg(row_of_pair + row * top + threadIdx.x)) * ldy;
-    }
+    __shared__ StagedPieces staged;
+    stage_pieces(pieces, row, staged);
     __syncthreads();
-    for (int c = threadIdx.x; c < width; c += 256) {
-        float sum = 0.0f;
-#pragma unroll 4
-        for (int j = 0; j < top; ++j) sum = fmaf(weight[j], __ldcg(y + from[j] + c), sum);
-        if (shared_y) {
-            const float v = mlr_load(shared_y + static_cast<size_t>(row) * ld_shared, c);
-            sum = shared_gate ? fmaf(__ldcg(shared_gate + row), v, sum) : sum + v;
-        }
-        out[static_cast<size_t>(row) * ldo + c] = sum;
+    constexpr int V = VEC ? 4 : 1;
+    for (int c = threadIdx.x * V; c < width; c += 256 * V) {
+        const float4 v = piece_sum<VEC>(pieces, staged, row, c);
+        float* o = out + static_cast<size_t>(row) * ldo + c;
+        if constexpr (VEC) *reinterpret_cast<float4*>(o) = v;
+        else *o = v.x;
     }
     mlr_grid_dependents_may_start();
 }
 
 }  // namespace
 
-// router: float32 [experts (+ 1 with has_gate), width]; correction: float32 [experts] or null; counts: int32 [experts], zero before
+// router: float32 [experts (+ 1 with has_gate), width]; correction: float32 [experts] or null; routed: how many of the experts are real
+// (the others, the last, are identity experts, whose chosen weights are summed up in identity [rows]); counts: int32 [routed], zero before
 // the call (`mlr_experts_arrange` zeroes them again).  chosen, place: int32 [rows, top]; weights: float32 [rows, top]; shared_gate [rows].
 MLR_API int mlr_experts_route(const void* x, long long ld, int act_bf16, const float* router, const float* correction, int rows, int width,
-                              int experts, int groups, int keep, int top, int has_gate, int* chosen, float* weights, int* place, int* counts,
-                              float* shared_gate, int kind, cudaStream_t stream) {
-    MLR_REQUIRE(kind == 0 || (kind == 1 && groups == 1), "experts_route: unknown kind of router %d (or one that has no groups)", kind);
+                              int experts, int routed, int groups, int keep, int top, int has_gate, int* chosen, float* weights, int* place,
+                              int* counts, float* shared_gate, float* identity, int kind, cudaStream_t stream) {
+    MLR_REQUIRE(kind == 0 || kind == 2 || (kind == 1 && groups == 1), "experts_route: unknown kind of router %d (or one that has no groups)", kind);
+    MLR_REQUIRE(routed >= 1 && routed <= experts && (routed == experts || identity), "experts_route: %d real experts of %d, or no room for the others' weights",
+                routed, experts);
     MLR_REQUIRE(x && router && chosen && weights && place && counts && width > 0, "experts_route: bad arguments");
     MLR_REQUIRE(experts >= 1 && experts <= kMaxExperts && top >= 1 && top <= kMaxTop && top <= experts, "experts_route: %d of %d experts (at most %d of %d)",
                 top, experts, kMaxTop, kMaxExperts);
@@ -460,11 +488,11 @@ MLR_API int mlr_experts_route(const void* x, long long ld, int act_bf16, const f
     if (act_bf16) {
         if (shared > 48 * 1024) cudaFuncSetAttribute(route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));
         mlr_launch((route_kernel<__nv_bfloat16>), dim3(rows), dim3(threads), shared, stream, static_cast<const __nv_bfloat16*>(x), ld, router,
-                   correction, width, experts, groups, keep, top, has_gate, chosen, weights, place, counts, shared_gate, kind);
+                   correction, width, experts, routed, groups, keep, top, has_gate, chosen, weights, place, counts, shared_gate, identity, kind);
     } else {
         if (shared > 48 * 1024) cudaFuncSetAttribute(route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));
         mlr_launch((route_kernel<float>), dim3(rows), dim3(threads), shared, stream, static_cast<const float*>(x), ld, router, correction, width,
-                   experts, groups, keep, top, has_gate, chosen, weights, place, counts, shared_gate, kind);
+                   experts, routed, groups, keep, top, has_gate, chosen, weights, place, counts, shared_gate, identity, kind);
     }
     return mlr_launched("experts_route");
 }
@@ -586,16 +614,17 @@ MLR_API int mlr_batched_product_bf16(const void* a, long long lda, const void* w
     return mlr_batched_product_bf16_strided(a, lda, K, w, out, ldo, N, rows, count, N, K, stream);
 }
 
-MLR_API int mlr_experts_combine(const float* y, long long ldy, const int* row_of_pair, const float* weights, int top, const void* shared_y,
-                                long long ld_shared, int shared_bf16, const float* shared_gate, float* out, long long ldo, int rows, int width,
-                                cudaStream_t stream) {
-    MLR_REQUIRE(y && row_of_pair && weights && out && top >= 1 && width > 0, "experts_combine: bad arguments");
+// out [rows, width] = the pieces added up (`Pieces`); shared (float32), gate, and x with identity may be null.
+MLR_API int mlr_experts_combine(const float* y, long long ldy, const int* row_of_pair, const float* weights, int top, const float* shared_y,
+                                long long ld_shared, const float* shared_gate, const void* x, long long ld_x, int x_bf16, const float* identity,
+                                float* out, long long ldo, int rows, int width, cudaStream_t stream) {
+    MLR_REQUIRE(y && out && width > 0, "experts_combine: bad arguments");
+    const Pieces pieces = {y, ldy, row_of_pair, weights, top, shared_y, ld_shared, shared_gate, x, ld_x, x_bf16, identity};
+    if (check_pieces(pieces, width, "experts_combine")) return 1;
     if (rows <= 0) return 0;
-    if (shared_bf16)
-        mlr_launch((combine_kernel<__nv_bfloat16>), dim3(rows), dim3(256), 0, stream, y, ldy, row_of_pair, weights, top,
-                   static_cast<const __nv_bfloat16*>(shared_y), ld_shared, shared_gate, out, ldo, width);
+    if (pieces_aligned(pieces) && width % 4 == 0 && ldo % 4 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0)
+        mlr_launch(combine_kernel<true>, dim3(rows), dim3(256), 0, stream, pieces, out, ldo, width);
     else
-        mlr_launch((combine_kernel<float>), dim3(rows), dim3(256), 0, stream, y, ldy, row_of_pair, weights, top,
-                   static_cast<const float*>(shared_y), ld_shared, shared_gate, out, ldo, width);
+        mlr_launch(combine_kernel<false>, dim3(rows), dim3(256), 0, stream, pieces, out, ldo, width);
     return mlr_launched("experts_combine");
 }

@@ -12,7 +12,9 @@
 //       delta:   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;      o = S^T q       (gated delta rule)
 //                with g = exp(-exp(a_log[head]) softplus(a + dt_bias[head])), beta = sigmoid(b), from two more
 //                columns of the projections' output per head
-//     Either rule may have a decay per head AND key channel instead (channel_decay): it acts on the rows of S, and comes from a
+//       step:    dt = softplus(a + dt_bias[head]);  S <- exp(-exp(a_log[head]) dt) S + dt k v^T;  o = S^T q + skip[head] v
+//                (state-space duality), from one more column of the projections' output per head
+//     Either of the first two rules may have a decay per head AND key channel instead (channel_decay): it acts on the rows of S, and comes from a
 //     product of small rank whose first half is among the projections (decay_rank columns of `side`):
 //         z = a W[decay_rank, heads * dim] + bias
 //         1: sigmoid(z)^(1 / tau)                            (gated linear attention)
@@ -21,18 +23,14 @@
 //   (q, k, v come from one buffer, `proj`; a, b and the gate from another, `side`, which may be the same)
 //   read-out:    o / sqrt(mean(o^2) + eps) per head, times a weight [vdim] (optional), times silu(gate)
 //                or sigmoid(gate) (optional), times a constant; with norm_all the root mean square is taken over
-//                the outputs of all heads of a token together and the weight is [heads * vdim]
+//                the outputs of all heads of a token together and the weight is [heads * vdim]; with gate_first the gate
+//                comes before the norm, which is taken over norm_parts equal parts of all heads' outputs side by side
 //
 // The columns of S are independent of one another in both rules, so a warp owns a few columns (lanes
 // split `dim`), and one block owns one (request, head): it prepares a batch of tokens in shared memory,
 // its warps walk the batch token by token, and the block norms and gates the batch's outputs.  The
 // state is read at the start and written at the end; a new request's state is zero (the caller zeroes
 // the slot).  Everything but the loads of the projections and the store of the result is float32.
-//
-// `mlr_short_conv` is the causal convolution over time per channel that precedes such a mixer in some
-// designs (taps [channels, n], the last tap is the current token's; silu after it), with the last n-1
-// inputs of every request kept as state; `mlr_short_conv_state` moves that state on after a step.  `mlr_short_conv_step` does both for
-// steps of few rows.
 #include "common.cuh"
 
 #include <type_traits>
@@ -43,12 +41,13 @@ struct RecurrenceSpec {
     const float* a_log;        // [heads] (rule 1)
     const float* dt_bias;      // [heads] (rule 1), or with channel_decay its bias [heads * dim]
     const float* out_weight;   // [vdim] or null
+    const float* skip;         // [heads] (rule 2)
     const void* decay_w;       // [decay_rank, heads * dim] in the activations' precision (channel_decay)
     const void* gate_w;        // [gate_rank, heads * vdim] in the activations' precision (gate_rank > 0)
     int heads, qk_heads, dim, vdim;
     int prep;                  // 0 none, 1 rotate, 2 unit
     int rot_dims;
-    int rule;                  // 0 decay, 1 delta
+    int rule;                  // 0 decay, 1 delta, 2 step
     int gate_kind;             // 0 none, 1 sigmoid, 2 silu
     int col_q, col_k, col_v;           // first columns of q, k, v in `proj`
     int col_a, col_b, col_gate;        // first columns of the rule's two inputs and of the gate in `side`
@@ -56,6 +55,7 @@ struct RecurrenceSpec {
     int norm_all;                      // 0: the read-out norms every head alone; 1: all heads of a token together
     int channel_decay;                 // 0: one decay per head; 1: sigmoid(z)^(1 / tau), 2: exp(-exp(a_log) softplus(z)) per key channel
     int decay_rank, gate_rank;         // columns of `side` from col_a on; from col_gate on (0: the gate itself is there)
+    int gate_first, norm_parts;        // gate_first: gate, then a norm over each of norm_parts equal parts of [heads * vdim], then the weight [heads * vdim]
     float q_mult, k_mult, unit_eps, eps, out_scale;
     float inv_tau;
 };
@@ -147,6 +147,11 @@ __global__ void __launch_bounds__(1024) linear_recurrence_kernel(const T* proj, 
             if (!CH) gs[threadIdx.x] = expf(-expf(s.a_log[head]) * softplus(mlr_load(row, s.col_a + head) + s.dt_bias[head]));
             bs[threadIdx.x] = 1.0f / (1.0f + expf(-b));
         }
+        if (s.rule == 2 && threadIdx.x < n) {
+            const float dt = softplus_exact(mlr_load(side + static_cast<size_t>(first + base + threadIdx.x) * ld_side, s.col_a + head) + s.dt_bias[head]);
+            gs[threadIdx.x] = expf(-expf(s.a_log[head]) * dt);
+            bs[threadIdx.x] = dt;
+        }
         if constexpr (CH) {
             const int ranks = s.decay_rank + s.gate_rank;
             for (int i = threadIdx.x; i < n * ranks; i += threads) {
@@ -215,14 +220,15 @@ __global__ void __launch_bounds__(1024) linear_recurrence_kernel(const T* proj, 
                     qq[r] = d < s.dim ? qs[static_cast<size_t>(t) * s.dim + d] : 0.0f;
                 }
                 float o[COLS];
-                if (s.rule == 0) {
+                if (s.rule != 1) {
+                    const float g = !CH && s.rule == 2 ? gs[t] : decay, write = !CH && s.rule == 2 ? bs[t] : 1.0f;
 #pragma unroll
                     for (int c = 0; c < COLS; ++c) {
-                        const float v = col0 + c < s.vdim ? vs[static_cast<size_t>(t) * s.vdim + col0 + c] : 0.0f;
+                        const float v = write * (col0 + c < s.vdim ? vs[static_cast<size_t>(t) * s.vdim + col0 + c] : 0.0f);
                         float dot = 0.0f;
 #pragma unroll
                         for (int r = 0; r < R; ++r) {
-                            S[c][r] = fmaf(CH ? dd[r] : decay, S[c][r], kk[r] * v);
+                            S[c][r] = fmaf(CH ? dd[r] : g, S[c][r], kk[r] * v);
                             dot = fmaf(S[c][r], qq[r], dot);
                         }
                         o[c] = dot;
@@ -270,7 +276,11 @@ __global__ void __launch_bounds__(1024) linear_recurrence_kernel(const T* proj, 
             const float* o = os + static_cast<size_t>(t) * s.vdim;
             if (raw) {
                 float* rrow = raw + (static_cast<size_t>(first + base + t) * s.heads + head) * s.vdim;
-                for (int c = lane; c < s.vdim; c += 32) rrow[c] = o[c];
+                if (!CH && s.rule == 2) {
+                    for (int c = lane; c < s.vdim; c += 32) rrow[c] = fmaf(s.skip[head], vs[static_cast<size_t>(t) * s.vdim + c], o[c]);
+                } else {
+                    for (int c = lane; c < s.vdim; c += 32) rrow[c] = o[c];
+                }
                 continue;
             }
             float inv = 1.0f;
@@ -309,7 +319,7 @@ __global__ void __launch_bounds__(1024) linear_recurrence_kernel(const T* proj, 
 // preparation and the read-out are parallel over rows, and the scan, the only sequential part, has a block per
 // (request, head, group of 16 columns of the state).
 
-// q and k of every row, prepared, as float32 [rows, qk_heads * dim] each; for the delta rule also g and beta [rows, 2 * heads].  zf
+// q and k of every row, prepared, as float32 [rows, qk_heads * dim] each; for the delta rule also g and beta, for the step rule g and dt [rows, 2 * heads].  zf
 // (or null): [rows, heads * dim], z of every key channel without its bias, turned into the channel's decay in place.
 constexpr int kPrepareThreads = 256;
 
@@ -361,6 +371,14 @@ __global__ void __launch_bounds__(kPrepareThreads) recurrence_prepare_kernel(con
             gates[static_cast<size_t>(row) * 2 * s.heads + s.heads + h] = 1.0f / (1.0f + expf(-b));
         }
     }
+    if (s.rule == 2) {
+        const T* sd = side + static_cast<size_t>(row) * ld_side;
+        for (int h = threadIdx.x; h < s.heads; h += blockDim.x) {
+            const float dt = softplus_exact(mlr_load(sd, s.col_a + h) + s.dt_bias[h]);
+            gates[static_cast<size_t>(row) * 2 * s.heads + h] = expf(-expf(s.a_log[h]) * dt);
+            gates[static_cast<size_t>(row) * 2 * s.heads + s.heads + h] = dt;
+        }
+    }
     if (zf) {
         const int channels = s.heads * s.dim;
         float* z = zf + static_cast<size_t>(row) * channels;
@@ -381,44 +399,6 @@ __global__ void __launch_bounds__(kPrepareThreads) recurrence_prepare_kernel(con
 // The second halves of the low-rank products of `kChannelRows` rows: df [rows, heads * dim] the decays, gf [rows, heads * vdim] the
 // read-out's gate before its sigmoid (gate_rank > 0).  A thread has one channel; the rows' small vectors stand in shared memory.
 constexpr int kChannelRows = 16, kChannelThreads = 128;
-
-// V neighbouring values as float32 (V = 1: any address; 4: an aligned group).
-template <int V, typename T>
-__device__ __forceinline__ void load_group(const T* p, float* v) {
-    if constexpr (V == 1) {
-        v[0] = mlr_load(p, 0);
-    } else if constexpr (sizeof(T) == 4) {
-#pragma unroll
-        for (int i = 0; i < V; i += 4) {
-            const float4 x = __ldcg(reinterpret_cast<const float4*>(p + i));
-            v[i] = x.x; v[i + 1] = x.y; v[i + 2] = x.z; v[i + 3] = x.w;
-        }
-    } else {
-#pragma unroll
-        for (int i = 0; i < V; i += 4) {
-            const uint2 x = __ldcg(reinterpret_cast<const uint2*>(p + i));
-            const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&x.x), hi = *reinterpret_cast<const __nv_bfloat162*>(&x.y);
-            const float2 f = __bfloat1622float2(lo), g = __bfloat1622float2(hi);
-            v[i] = f.x; v[i + 1] = f.y; v[i + 2] = g.x; v[i + 3] = g.y;
-        }
-    }
-}
-
-template <int V, typename T>
-__device__ __forceinline__ void store_group(T* p, const float* v) {
-    if constexpr (V == 1) {
-        mlr_store(p, 0, v[0]);
-    } else if constexpr (sizeof(T) == 4) {
-#pragma unroll
-        for (int i = 0; i < V; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
-    } else {
-#pragma unroll
-        for (int i = 0; i < V; i += 4) {
-            const __nv_bfloat162 lo = __floats2bfloat162_rn(v[i], v[i + 1]), hi = __floats2bfloat162_rn(v[i + 2], v[i + 3]);
-            *reinterpret_cast<uint2*>(p + i) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
-        }
-    }
-}
 
 // V channels a thread (V = 4 where every row of the second matrices starts on a border of four values).
 template <typename T, int V>
@@ -458,19 +438,19 @@ __global__ void __launch_bounds__(kChannelThreads) recurrence_channel_kernel(con
         for (; r + kAhead <= rank; r += kAhead) {
             float v[kAhead][V];
 #pragma unroll
-            for (int i = 0; i < kAhead; ++i) load_group<V>(w + static_cast<size_t>(r + i) * width, v[i]);
+            for (int i = 0; i < kAhead; ++i) mlr_load_group<V>(w + static_cast<size_t>(r + i) * width, v[i]);
 #pragma unroll
             for (int i = 0; i < kAhead; ++i) add(r + i, v[i]);
         }
         for (; r < rank; ++r) {
             float v[V];
-            load_group<V>(w + static_cast<size_t>(r) * width, v);
+            mlr_load_group<V>(w + static_cast<size_t>(r) * width, v);
             add(r, v);
         }
         // The decays' functions are long: they stand once, in a loop over the rows, whose sums wait in shared memory.
         float* zs = lows + rank_room * kChannelRows + threadIdx.x * V;        // [kChannelRows][threads * V], a thread's own columns
 #pragma unroll
-        for (int t = 0; t < kChannelRows; ++t) store_group<V>(zs + t * kPerBlock, acc[t]);
+        for (int t = 0; t < kChannelRows; ++t) mlr_store_group<V>(zs + t * kPerBlock, acc[t]);
         float* out = (is_gate ? gf : df) + static_cast<size_t>(row0) * width + c;
         float bias[V] = {};
         if (!is_gate) {
@@ -486,7 +466,7 @@ __global__ void __launch_bounds__(kChannelThreads) recurrence_channel_kernel(con
 #pragma unroll
                 for (int j = 0; j < V; ++j) z[j] = channel_decay_of(s, z[j] + bias[j], (c + j) / s.dim);
             }
-            store_group<V>(out + static_cast<size_t>(t) * width, z);
+            mlr_store_group<V>(out + static_cast<size_t>(t) * width, z);
         }
     }
     mlr_grid_dependents_may_start();
@@ -563,7 +543,7 @@ __global__ void __launch_bounds__(kScanWarps * 32) recurrence_scan_kernel(const 
             const int t = i / kScanBlockCols, c = block_col + i % kScanBlockCols;
             v_next[j] = (t < n && c < s.vdim) ? mlr_load(proj + static_cast<size_t>(first + base + t) * ld, s.col_v + head * s.vdim + c) : 0.0f;
         }
-        if (s.rule == 1 && threadIdx.x < n) {
+        if (s.rule != 0 && threadIdx.x < n) {
             if constexpr (!CH) g_next = __ldcg(gates + static_cast<size_t>(first + base + threadIdx.x) * 2 * s.heads + head);
             b_next = __ldcg(gates + static_cast<size_t>(first + base + threadIdx.x) * 2 * s.heads + s.heads + head);
         }
@@ -599,14 +579,15 @@ __global__ void __launch_bounds__(kScanWarps * 32) recurrence_scan_kernel(const 
                 qq[r] = d < s.dim ? qnow[static_cast<size_t>(t) * s.dim + d] : 0.0f;
             }
             float o[kScanCols];
-            if (s.rule == 0) {
+            if (s.rule != 1) {
+                const float g = !CH && s.rule == 2 ? gs[t] : decay, write = !CH && s.rule == 2 ? bs[t] : 1.0f;
 #pragma unroll
                 for (int c = 0; c < kScanCols; ++c) {
-                    const float v = vs[t * kScanBlockCols + warp * kScanCols + c];
+                    const float v = write * vs[t * kScanBlockCols + warp * kScanCols + c];
                     float dot = 0.0f;
 #pragma unroll
                     for (int r = 0; r < R; ++r) {
-                        S[c][r] = fmaf(CH ? dd[r] : decay, S[c][r], kk[r] * v);
+                        S[c][r] = fmaf(CH ? dd[r] : g, S[c][r], kk[r] * v);
                         dot = fmaf(S[c][r], qq[r], dot);
                     }
                     o[c] = dot;
@@ -649,7 +630,8 @@ __global__ void __launch_bounds__(kScanWarps * 32) recurrence_scan_kernel(const 
         __syncthreads();
         for (int i = threadIdx.x; i < n * kScanBlockCols; i += blockDim.x) {
             const int t = i / kScanBlockCols, c = block_col + i % kScanBlockCols;
-            if (c < s.vdim) obuf[static_cast<size_t>(first + base + t) * o_ld + static_cast<size_t>(head) * s.vdim + c] = os[i];
+            const float o = !CH && s.rule == 2 ? fmaf(s.skip[head], vs[i], os[i]) : os[i];
+            if (c < s.vdim) obuf[static_cast<size_t>(first + base + t) * o_ld + static_cast<size_t>(head) * s.vdim + c] = o;
         }
     }
     mlr_grid_dependents_may_start();     // only now: blocks of the next grid that wait on this SM slow the walk
@@ -726,7 +708,7 @@ __global__ void __launch_bounds__(kColumnWarps * 32) recurrence_scan16_kernel(co
             const int t = i / kScanBlockCols, c = block_col + i % kScanBlockCols;
             v_next[j] = proj[(t < n && c < s.vdim) ? static_cast<size_t>(first + base + t) * ld + s.col_v + head * s.vdim + c : 0];
         }
-        if (RULE == 1 && threadIdx.x < n) {
+        if (RULE != 0 && threadIdx.x < n) {
             const float* g = gates + static_cast<size_t>(first + base + threadIdx.x) * 2 * s.heads + head;
             if constexpr (!CH) g_next = __ldcg(g);
             b_next = __ldcg(g + s.heads);
@@ -746,7 +728,7 @@ __global__ void __launch_bounds__(kColumnWarps * 32) recurrence_scan16_kernel(co
             const int i = threadIdx.x + j * kThreads;
             if (i < batch * kScanBlockCols) vs[i % kScanBlockCols * batch + i / kScanBlockCols] = act_in(mlr_load(&v_next[j], 0), s.in_act);
         }
-        if (RULE == 1 && threadIdx.x < batch) {
+        if (RULE != 0 && threadIdx.x < batch) {
             gs[threadIdx.x] = g_next;
             bs[threadIdx.x] = b_next;
         }
@@ -781,7 +763,7 @@ __global__ void __launch_bounds__(kColumnWarps * 32) recurrence_scan16_kernel(co
             const float4 v4 = *reinterpret_cast<const float4*>(vs + my_col * batch + t0);
             const float v[4] = {v4.x, v4.y, v4.z, v4.w};
             [[maybe_unused]] float g[4] = {decay, decay, decay, decay}, beta[4] = {};
-            if constexpr (RULE == 1) {
+            if constexpr (RULE != 0) {
                 const float4 b4 = *reinterpret_cast<const float4*>(bs + t0);
                 beta[0] = b4.x; beta[1] = b4.y; beta[2] = b4.z; beta[3] = b4.w;
                 if constexpr (!CH) {
@@ -796,8 +778,8 @@ __global__ void __launch_bounds__(kColumnWarps * 32) recurrence_scan16_kernel(co
                 if (!kGuarded || t0 + u < n) {
                     const Token& x = tokens[u & 1];
                     load(tokens[(u + 1) & 1], u < 3 && !kGuarded ? t0 + u + 1 : min(t0 + u + 1, n - 1));
-                    float write = v[u];
-                    if constexpr (RULE == 0) {
+                    float write = RULE == 2 ? beta[u] * v[u] : v[u];
+                    if constexpr (RULE != 1) {
 #pragma unroll
                         for (int j = 0; j < E; ++j) S[j] = fmaf(CH ? x.d[CH ? j : 0] : g[u], S[j], x.k[j] * write);
                     } else {
@@ -836,7 +818,8 @@ __global__ void __launch_bounds__(kColumnWarps * 32) recurrence_scan16_kernel(co
         __syncthreads();
         for (int i = threadIdx.x; i < n * kScanBlockCols; i += kThreads) {
             const int t = i / kScanBlockCols, c = block_col + i % kScanBlockCols;
-            if (c < s.vdim) obuf[static_cast<size_t>(first + base + t) * o_ld + static_cast<size_t>(head) * s.vdim + c] = os[i];
+            const float o = RULE == 2 ? fmaf(s.skip[head], vs[i % kScanBlockCols * batch + t], os[i]) : os[i];
+            if (c < s.vdim) obuf[static_cast<size_t>(first + base + t) * o_ld + static_cast<size_t>(head) * s.vdim + c] = o;
         }
     }
     mlr_grid_dependents_may_start();     // only now: blocks of the next grid that wait on this SM slow the walk
@@ -877,7 +860,7 @@ __global__ void __launch_bounds__(kReadoutThreads) recurrence_readout_kernel(con
 #pragma unroll
         for (int i = 0; i < kHeld; ++i) {
             const int c = (i * 32 + lane) * V;
-            if (c < s.vdim) load_group<V>(o + c, held[i]);
+            if (c < s.vdim) mlr_load_group<V>(o + c, held[i]);
         }
         float inv = inv_all;
         if (s.eps >= 0.0f && !s.norm_all) {
@@ -899,8 +882,8 @@ __global__ void __launch_bounds__(kReadoutThreads) recurrence_readout_kernel(con
             if (c >= s.vdim) break;
             float g[V] = {};
             if (s.gate_kind) {
-                if (gf) load_group<V>(gfrow + c, g);
-                else load_group<V>(grow + c, g);
+                if (gf) mlr_load_group<V>(gfrow + c, g);
+                else mlr_load_group<V>(grow + c, g);
             }
             float value[V];
 #pragma unroll
@@ -913,109 +896,62 @@ __global__ void __launch_bounds__(kReadoutThreads) recurrence_readout_kernel(con
                 }
                 value[j] *= s.out_scale;
             }
-            store_group<V>(orow + c, value);
+            mlr_store_group<V>(orow + c, value);
         }
     }
     mlr_grid_dependents_may_start();
 }
 
-constexpr int kMaxTaps = 16;
-constexpr int kConvRows = 8, kConvThreads = 128;
-
-// A thread has V neighbouring channels and walks rows with the last taps - 1 inputs in registers.  N: the number of taps, or 0 for any
-// number (then V = 1).  STEP: a block has a segment's rows, all of them, and moves the segment's state on behind them; else it has
-// kConvRows rows of the batch, whatever their segments, and the state is read only.
-template <typename T, int V, int N, bool STEP>
-__global__ void __launch_bounds__(kConvThreads) short_conv_kernel(const T* in, int ld_in, T* out, int ld_out, int channels, int taps,
-                                                                  const float* weights, float* state, long long state_stride,
-                                                                  const int* segment_info, const int* segment_of_row, int rows) {
+// The read-out with the gate in front: o times its gate (`side`), each of s.norm_parts equal parts of a token's outputs (all heads side
+// by side) over its own root mean square, times the weight [heads * vdim] and the constant.  A block per row, the gated values in
+// shared memory: [heads * vdim] and one sum per part.
+template <typename T, int V>
+__global__ void __launch_bounds__(kReadoutThreads) recurrence_parts_readout_kernel(const float* obuf, const T* side, int ld_side, T* out, int ld_out,
+                                                                                  RecurrenceSpec s) {
     mlr_grid_wait();
-    constexpr int kBack = (N ? N : kMaxTaps) - 1;
-    const int back = N ? N - 1 : taps - 1;
-    const int c = (blockIdx.y * kConvThreads + threadIdx.x) * V;
-    if (c >= channels) return;
-    float w[kBack + 1][V], past[kBack + 1][V];                  // past[i]: the input that tap i sees
+    extern __shared__ __align__(16) float gated[];
+    __shared__ float scratch[32];
+    const int row = blockIdx.x, total = s.heads * s.vdim, part = total / s.norm_parts;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    float* inv = gated + (total + 3) / 4 * 4;
+    const float* o = obuf + static_cast<size_t>(row) * total;
+    const T* grow = side + static_cast<size_t>(row) * ld_side + s.col_gate;
+    float mine = 0.0f;
+    for (int c = threadIdx.x * V; c < total; c += blockDim.x * V) {
+        float v[V], g[V];
+        mlr_load_group<V>(o + c, v);
+        if (s.gate_kind) {
+            mlr_load_group<V>(grow + c, g);
 #pragma unroll
-    for (int i = 0; i <= kBack; ++i)
-#pragma unroll
-        for (int j = 0; j < V; ++j) w[i][j] = i <= back ? weights[static_cast<size_t>(c + j) * (back + 1) + i] : 0.0f;
-    int row = STEP ? segment_info[4 * blockIdx.x] : blockIdx.x * kConvRows;
-    const int end = STEP ? row + segment_info[4 * blockIdx.x + 1] : min(row + kConvRows, rows);
-    int segment = -1;
-    float next[V];
-    if (row < end) load_group<V>(in + static_cast<size_t>(row) * ld_in + c, next);
-    float* mine = nullptr;
-    for (; row < end; ++row) {
-        const int now = STEP ? static_cast<int>(blockIdx.x) : segment_of_row[row];
-        if (now != segment) {                                   // the inputs before this row: of this step, or from the state
-            segment = now;
-            const int first = segment_info[4 * segment], j0 = row - first;
-            mine = state + static_cast<size_t>(segment_info[4 * segment + 3]) * state_stride + c;
-#pragma unroll
-            for (int i = 0; i < kBack; ++i)
-                if (i < back) {
-                    const int m = j0 - back + i;
-                    if (m >= 0) load_group<V>(in + static_cast<size_t>(first + m) * ld_in + c, past[i]);
-                    else {
-#pragma unroll
-                        for (int j = 0; j < V; ++j) past[i][j] = mine[static_cast<size_t>(back + m) * channels + j];
-                    }
-                }
+            for (int j = 0; j < V; ++j) {
+                const float sig = 1.0f / (1.0f + expf(-g[j]));
+                v[j] *= s.gate_kind == 2 ? g[j] * sig : sig;
+            }
         }
-        float x[V], y[V] = {};
 #pragma unroll
-        for (int j = 0; j < V; ++j) x[j] = next[j];
-        if (row + 1 < end) load_group<V>(in + static_cast<size_t>(row + 1) * ld_in + c, next);
-#pragma unroll
-        for (int i = 0; i < kBack; ++i)
-            if (i < back) {
-#pragma unroll
-                for (int j = 0; j < V; ++j) y[j] = fmaf(w[i][j], past[i][j], y[j]);
-            }
-#pragma unroll
-        for (int i = 0; i <= kBack; ++i)
-            if (i == back) {
-#pragma unroll
-                for (int j = 0; j < V; ++j) y[j] = fmaf(w[i][j], x[j], y[j]);
-            }
-#pragma unroll
-        for (int j = 0; j < V; ++j) y[j] = y[j] / (1.0f + expf(-y[j]));
-        store_group<V>(out + static_cast<size_t>(row) * ld_out + c, y);
-#pragma unroll
-        for (int i = 0; i < kBack; ++i)
-            if (i < back) {
-#pragma unroll
-                for (int j = 0; j < V; ++j) past[i][j] = i + 1 < back ? past[i + 1][j] : x[j];
-            }
+        for (int j = 0; j < V; ++j) mine = fmaf(v[j], v[j], mine);
+        mlr_store_group<V>(gated + c, v);
     }
-    if constexpr (STEP) {
-        if (mine) {
-#pragma unroll
-            for (int i = 0; i < kBack; ++i)
-                if (i < back) {
-#pragma unroll
-                    for (int j = 0; j < V; ++j) mine[static_cast<size_t>(i) * channels + j] = past[i][j];
-                }
+    if (s.norm_parts == 1) {
+        const float sum = mlr_block_sum(mine, scratch);
+        if (threadIdx.x == 0) inv[0] = 1.0f / sqrtf(sum / static_cast<float>(part) + s.eps);
+        __syncthreads();
+    } else {
+        __syncthreads();
+        for (int g = warp; g < s.norm_parts; g += warps) {
+            float sum = 0.0f;
+            for (int c = lane; c < part; c += 32) sum = fmaf(gated[g * part + c], gated[g * part + c], sum);
+            sum = mlr_warp_sum(sum);
+            if (lane == 0) inv[g] = 1.0f / sqrtf(sum / static_cast<float>(part) + s.eps);
         }
+        __syncthreads();
     }
-    mlr_grid_dependents_may_start();
-}
-
-template <typename T>
-__global__ void __launch_bounds__(256) short_conv_state_kernel(const T* in, int ld_in, int channels, int taps, float* state,
-                                                               long long state_stride, const int* segment_info) {
-    mlr_grid_wait();
-    const int segment = blockIdx.x;
-    const int first = segment_info[4 * segment], count = segment_info[4 * segment + 1], slot = segment_info[4 * segment + 3];
-    float* mine = state + static_cast<size_t>(slot) * state_stride;
-    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < channels; c += gridDim.y * blockDim.x) {
-        float kept[kMaxTaps];
-        for (int i = 0; i < taps - 1; ++i) kept[i] = mine[static_cast<size_t>(i) * channels + c];
-        for (int i = 0; i < taps - 1; ++i) {
-            const int m = count - (taps - 1) + i;
-            mine[static_cast<size_t>(i) * channels + c] =
-                m >= 0 ? mlr_load(in + static_cast<size_t>(first + m) * ld_in, c) : kept[taps - 1 + m];
-        }
+    T* orow = out + static_cast<size_t>(row) * ld_out;
+    for (int c = threadIdx.x * V; c < total; c += blockDim.x * V) {
+        float v[V];
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[j] = gated[c + j] * inv[(c + j) / part] * (s.out_weight ? s.out_weight[c + j] : 1.0f) * s.out_scale;
+        mlr_store_group<V>(orow + c, v);
     }
     mlr_grid_dependents_may_start();
 }
@@ -1031,7 +967,12 @@ static int check_recurrence(const RecurrenceSpec& s) {
                 "linear_recurrence: a state of %d x %d per head is more than a block's registers hold (256 x 128 or 128 x 256)", s.dim, s.vdim);
     MLR_REQUIRE(s.prep != 1 || (s.rot_dims >= 0 && s.rot_dims % 2 == 0 && s.rot_dims <= s.dim && (s.rot_dims == 0 || s.freq)),
                 "linear_recurrence: %d rotated values do not fit a head of %d", s.rot_dims, s.dim);
-    MLR_REQUIRE(s.rule == 0 || s.rule == 1, "linear_recurrence: no rule %d", s.rule);
+    MLR_REQUIRE(s.rule >= 0 && s.rule <= 2, "linear_recurrence: no rule %d", s.rule);
+    MLR_REQUIRE(s.rule != 2 || (s.skip && !s.channel_decay && s.gate_first), "linear_recurrence: the step rule goes with a skip per head and the gate before the norm");
+    MLR_REQUIRE(!s.gate_first || (s.norm_parts >= 1 && (s.heads * s.vdim) % s.norm_parts == 0 && !s.gate_rank && s.eps >= 0.0f),
+                "linear_recurrence: %d values of all heads cannot be normed in %d parts", s.heads * s.vdim, s.norm_parts);
+    MLR_REQUIRE(!s.gate_first || sizeof(float) * (static_cast<size_t>(s.heads) * s.vdim + s.norm_parts + 4) <= 200 * 1024,
+                "linear_recurrence: %d values of all heads do not fit shared memory", s.heads * s.vdim);
     if (s.channel_decay) {
         MLR_REQUIRE((s.channel_decay == 1 || (s.channel_decay == 2 && s.a_log)) && s.dt_bias && s.decay_w && s.decay_rank >= 1 &&
                         s.decay_rank <= kMaxRank, "linear_recurrence: a decay per channel needs its product (rank 1 to %d) and its constants", kMaxRank);
@@ -1048,6 +989,16 @@ template <typename T>
 void launch_readout(const RecurrenceSpec& s, const float* obuf, const T* side, int ld_side, const float* gf, T* out, int ld_out, int rows,
                     cudaStream_t stream) {
     const auto aligned = [](const void* p, size_t bytes) { return reinterpret_cast<uintptr_t>(p) % bytes == 0; };
+    if (s.gate_first) {
+        const int total = s.heads * s.vdim;
+        const size_t shared = sizeof(float) * ((total + 3) / 4 * 4 + s.norm_parts);
+        const bool four = total % 4 == 0 && aligned(obuf, 16) && aligned(out, 4 * sizeof(T)) && ld_out % 4 == 0 &&
+                          (!s.gate_kind || (aligned(side + s.col_gate, 4 * sizeof(T)) && ld_side % 4 == 0));
+        const auto kernel = four ? recurrence_parts_readout_kernel<T, 4> : recurrence_parts_readout_kernel<T, 1>;
+        if (shared > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));
+        mlr_launch(kernel, dim3(rows), dim3(kReadoutThreads), shared, stream, obuf, side, ld_side, out, ld_out, s);
+        return;
+    }
     // Head sizes that are no multiple of 32 keep the one-kernel form's order of every sum (the same bits in both forms).
     const bool vec = s.dim % 32 == 0 && s.vdim % 4 == 0 && aligned(obuf, 16) && aligned(out, 4 * sizeof(T)) && ld_out % 4 == 0 &&
                      (!s.gate_kind || (gf ? aligned(gf, 16) : aligned(side + s.col_gate, 4 * sizeof(T)) && ld_side % 4 == 0));
@@ -1066,7 +1017,7 @@ MLR_API int mlr_linear_recurrence(const RecurrenceSpec* spec, const void* proj, 
     const RecurrenceSpec& s = *spec;
     if (check_recurrence(s)) return 1;
     MLR_REQUIRE(n_segments >= 0 && state && proj && side && out, "linear_recurrence: bad arguments");
-    MLR_REQUIRE(!s.norm_all || obuf, "linear_recurrence: a norm over all heads needs the buffer of plain outputs");
+    MLR_REQUIRE(!(s.norm_all || s.gate_first) || obuf, "linear_recurrence: a norm over all heads needs the buffer of plain outputs");
     MLR_REQUIRE(!s.gate_rank || !obuf, "linear_recurrence: plain outputs have no place for a low-rank gate");
     if (n_segments == 0) return 0;
     const int cols = s.vdim > 128 ? 8 : 4;
@@ -1112,7 +1063,7 @@ MLR_API int mlr_linear_recurrence(const RecurrenceSpec* spec, const void* proj, 
     return mlr_launched("linear_recurrence");
 }
 
-// The three-kernel form.  qf, kf: float32 [rows, qk_heads * dim]; gates: float32 [rows, 2 * heads] (delta rule; else unused);
+// The three-kernel form.  qf, kf: float32 [rows, qk_heads * dim]; gates: float32 [rows, 2 * heads] (delta and step rules; else unused);
 // obuf: float32 [rows, heads * vdim].  Same results as `mlr_linear_recurrence` up to the order in which a column's sums are added
 // (the same order for head sizes that are no multiple of 32).  With a decay per channel, df [rows, heads * dim] and (low-rank gate) gf
 // [rows, heads * vdim] are float32 room; with `products_made` they hold the low-rank products' results already (df without the bias).
@@ -1150,6 +1101,7 @@ MLR_API int mlr_linear_recurrence_split(const RecurrenceSpec* spec, const void* 
 #define MLR_COLUMN(T, DIM, CH)                                                                                                         \
     do {                                                                                                                               \
         if (s.rule == 0) MLR_WALK((recurrence_scan16_kernel<T, DIM, 0, CH>), T, kColumnWarps);                                         \
+        else if (s.rule == 2) MLR_WALK((recurrence_scan16_kernel<T, DIM, 2, false>), T, kColumnWarps);                                 \
         else MLR_WALK((recurrence_scan16_kernel<T, DIM, 1, CH>), T, kColumnWarps);                                                     \
     } while (0)
 #define MLR_SCAN(T, CH)                                                                                                                \
@@ -1192,65 +1144,4 @@ MLR_API int mlr_linear_recurrence_split(const RecurrenceSpec* spec, const void* 
 #undef MLR_COLUMN
 #undef MLR_WALK
     return mlr_launched("linear_recurrence_split");
-}
-
-namespace {
-template <bool STEP>
-int short_conv(const void* in, int ld_in, void* out, int ld_out, int act_bf16, int channels, int taps, const float* weights, float* state,
-               long long state_stride, const int* segment_info, const int* segment_of_row, int blocks, int rows, cudaStream_t stream) {
-    const size_t group_bytes = act_bf16 ? 8 : 16;
-    const bool wide = taps <= 4 && channels % 4 == 0 && ld_in % 4 == 0 && ld_out % 4 == 0 && reinterpret_cast<uintptr_t>(in) % group_bytes == 0 &&
-                      reinterpret_cast<uintptr_t>(out) % group_bytes == 0;
-    const dim3 grid(blocks, (channels + kConvThreads * (wide ? 4 : 1) - 1) / (kConvThreads * (wide ? 4 : 1)));
-#define MLR_CONV(T, V, N)                                                                                                              \
-    mlr_launch((short_conv_kernel<T, V, N, STEP>), dim3(grid), dim3(kConvThreads), 0, stream, static_cast<const T*>(in), ld_in,        \
-               static_cast<T*>(out), ld_out, channels, taps, weights, state, state_stride, segment_info, segment_of_row, rows)
-#define MLR_CONVS(T)                                                                                                                   \
-    do {                                                                                                                               \
-        if (!wide) MLR_CONV(T, 1, 0);                                                                                                  \
-        else if (taps == 1) MLR_CONV(T, 4, 1);                                                                                         \
-        else if (taps == 2) MLR_CONV(T, 4, 2);                                                                                         \
-        else if (taps == 3) MLR_CONV(T, 4, 3);                                                                                         \
-        else MLR_CONV(T, 4, 4);                                                                                                        \
-    } while (0)
-    if (act_bf16) MLR_CONVS(__nv_bfloat16);
-    else MLR_CONVS(float);
-#undef MLR_CONVS
-#undef MLR_CONV
-    return mlr_launched("short_conv");
-}
-}  // namespace
-
-MLR_API int mlr_short_conv(const void* in, int ld_in, void* out, int ld_out, int act_bf16, int channels, int taps,
-                           const float* weights, const float* state, long long state_stride, const int* segment_info,
-                           const int* segment_of_row, int rows, cudaStream_t stream) {
-    MLR_REQUIRE(channels > 0 && taps >= 1 && taps <= kMaxTaps, "short_conv: %d taps are outside [1, %d]", taps, kMaxTaps);
-    MLR_REQUIRE(ld_in >= channels && ld_out >= channels && (taps == 1 || state), "short_conv: bad strides or no state");
-    if (rows <= 0) return 0;
-    return short_conv<false>(in, ld_in, out, ld_out, act_bf16, channels, taps, weights, const_cast<float*>(state), state_stride, segment_info,
-                             segment_of_row, (rows + kConvRows - 1) / kConvRows, rows, stream);
-}
-
-// The convolution and the state behind it in one launch: a block walks all rows of a segment (steps of few rows).
-MLR_API int mlr_short_conv_step(const void* in, int ld_in, void* out, int ld_out, int act_bf16, int channels, int taps, const float* weights,
-                                float* state, long long state_stride, const int* segment_info, int n_segments, cudaStream_t stream) {
-    MLR_REQUIRE(channels > 0 && taps >= 1 && taps <= kMaxTaps, "short_conv_step: %d taps are outside [1, %d]", taps, kMaxTaps);
-    MLR_REQUIRE(ld_in >= channels && ld_out >= channels && (taps == 1 || state), "short_conv_step: bad strides or no state");
-    if (n_segments <= 0) return 0;
-    return short_conv<true>(in, ld_in, out, ld_out, act_bf16, channels, taps, weights, state, state_stride, segment_info, nullptr, n_segments, 0,
-                            stream);
-}
-
-MLR_API int mlr_short_conv_state(const void* in, int ld_in, int act_bf16, int channels, int taps, float* state,
-                                 long long state_stride, const int* segment_info, int n_segments, cudaStream_t stream) {
-    MLR_REQUIRE(channels > 0 && taps >= 1 && taps <= kMaxTaps, "short_conv_state: %d taps are outside [1, %d]", taps, kMaxTaps);
-    if (n_segments <= 0 || taps == 1) return 0;
-    const dim3 grid(n_segments, (channels + 255) / 256);
-    if (act_bf16)
-        mlr_launch((short_conv_state_kernel<__nv_bfloat16>), dim3(grid), dim3(256), 0, stream, static_cast<const __nv_bfloat16*>(in), ld_in,
-                   channels, taps, state, state_stride, segment_info);
-    else
-        mlr_launch((short_conv_state_kernel<float>), dim3(grid), dim3(256), 0, stream, static_cast<const float*>(in), ld_in, channels,
-                   taps, state, state_stride, segment_info);
-    return mlr_launched("short_conv_state");
 }

@@ -14,6 +14,7 @@
 //   The token before a row is the row above it, or, for the first row of a step's segment, what the
 //   request's state slot holds; the slot then takes the segment's last token.
 #include "common.cuh"
+#include "pieces.cuh"
 
 namespace {
 
@@ -31,14 +32,17 @@ struct StreamWeights {
 template <typename TO, int S, int V>
 __global__ void __launch_bounds__(kThreads) streams_step_kernel(float* h, const float* y, long long ld_y, const float* y_scale, const float* mix,
                                                                  const float* w_out, const float* w_in, const float* norm_weight, float eps,
-                                                                 TO* out, long long ld_out, const int* rows, int width, int streams_given) {
+                                                                 TO* out, long long ld_out, const int* rows, int width, int streams_given, Pieces pieces) {
     mlr_grid_wait();
+    __shared__ StagedPieces staged;
     extern __shared__ __align__(16) float u[];          // [width]
     __shared__ float scratch[32];
     __shared__ StreamWeights w;
     constexpr int kCopies = S ? S : kMaxStreams;
     const int streams = S ? S : streams_given;
     const int row = rows ? rows[blockIdx.x] : blockIdx.x;
+    const bool writes = y || pieces.y;
+    if (pieces.y) stage_pieces(pieces, row, staged);
     if (threadIdx.x < streams * streams && mix) w.mix[threadIdx.x] = mix[threadIdx.x];
     if (threadIdx.x < streams) {
         if (w_out) w.out[threadIdx.x] = w_out[threadIdx.x];
@@ -49,10 +53,10 @@ __global__ void __launch_bounds__(kThreads) streams_step_kernel(float* h, const 
     float rmix[S ? S * S : 1], rout[S ? S : 1], rin[S ? S : 1];
     if (S) {
 #pragma unroll
-        for (int i = 0; i < S * S; ++i) rmix[i] = y ? w.mix[i] : 0.0f;
+        for (int i = 0; i < S * S; ++i) rmix[i] = writes ? w.mix[i] : 0.0f;
 #pragma unroll
         for (int i = 0; i < S; ++i) {
-            rout[i] = y ? w.out[i] : 0.0f;
+            rout[i] = writes ? w.out[i] : 0.0f;
             rin[i] = w.in[i];
         }
     }
@@ -75,12 +79,19 @@ __global__ void __launch_bounds__(kThreads) streams_step_kernel(float* h, const 
         float sum[V];
 #pragma unroll
         for (int e = 0; e < V; ++e) sum[e] = 0.0f;
-        if (yrow) {
+        if (writes) {
             float add[V];
+            if (yrow) {
 #pragma unroll
-            for (int e = 0; e < V; ++e) {
-                add[e] = __ldcg(yrow + c + e);
-                if (y_scale) add[e] *= y_scale[c + e];
+                for (int e = 0; e < V; ++e) add[e] = __ldcg(yrow + c + e);
+            } else {
+                const float4 v = piece_sum<V == 4>(pieces, staged, row, c);
+                add[0] = v.x;
+                if (V == 4) add[V > 1 ? 1 : 0] = v.y, add[V > 2 ? 2 : 0] = v.z, add[V - 1] = v.w;
+            }
+            if (y_scale) {
+#pragma unroll
+                for (int e = 0; e < V; ++e) add[e] *= y_scale[c + e];
             }
 #pragma unroll
             for (int t = 0; t < kCopies; ++t) {
@@ -182,22 +193,25 @@ __global__ void __launch_bounds__(kThreads) embed_hashed_kernel(float* h, const 
 // optionally y_scale [width]: the write.  out (bfloat16 or float32 [count, width]) with norm_weight [width] (or null) and w_in
 // [streams] (or null: the plain sum): the read.  rows: which rows of h the `count` blocks work on (null: 0 .. count-1); with
 // `rows` the write must be absent (it would leave the other rows behind).
-MLR_API int mlr_streams_step(float* h, const float* y, long long ld_y, const float* y_scale, const float* mix, const float* w_out,
-                             const float* w_in, const float* norm_weight, float eps, void* out, long long ld_out, int out_bf16,
-                             const int* rows, int count, int width, int streams, cudaStream_t stream) {
+namespace {
+int streams_step(float* h, const float* y, long long ld_y, const float* y_scale, const float* mix, const float* w_out, const float* w_in,
+                 const float* norm_weight, float eps, void* out, long long ld_out, int out_bf16, const int* rows, int count, int width, int streams,
+                 const Pieces& pieces, cudaStream_t stream) {
     MLR_REQUIRE(h && width > 0 && streams >= 1 && streams <= kMaxStreams, "streams_step: 1 to %d copies of the stream, got %d", kMaxStreams, streams);
-    MLR_REQUIRE(y || out, "streams_step: neither a write nor a read");
-    MLR_REQUIRE(!y || (mix && w_out && !rows), "streams_step: a write needs its weights and all rows");
+    MLR_REQUIRE(y || out || pieces.y, "streams_step: neither a write nor a read");
+    MLR_REQUIRE(!(y || pieces.y) || (mix && w_out && !rows), "streams_step: a write needs its weights and all rows");
+    MLR_REQUIRE(!(y && pieces.y), "streams_step: a contribution in pieces stands instead of a plain one");
+    if (pieces.y && check_pieces(pieces, width, "streams_step")) return 1;
     MLR_REQUIRE(static_cast<size_t>(width) * sizeof(float) <= 200 * 1024, "streams_step: a width of %d does not fit shared memory", width);
     if (count <= 0) return 0;
     const size_t shared = out ? static_cast<size_t>(width) * sizeof(float) : 0;
-    const bool wide = width % 4 == 0 && reinterpret_cast<uintptr_t>(h) % 16 == 0;
+    const bool wide = width % 4 == 0 && reinterpret_cast<uintptr_t>(h) % 16 == 0 && (!pieces.y || pieces_aligned(pieces));
 #define MLR_GO(TO, S, V)                                                                                                                   \
     do {                                                                                                                                   \
         if (shared > 48 * 1024)                                                                                                            \
             cudaFuncSetAttribute(streams_step_kernel<TO, S, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));    \
         mlr_launch((streams_step_kernel<TO, S, V>), dim3(count), dim3(kThreads), shared, stream, h, y, ld_y, y_scale, mix, w_out, w_in,    \
-                   norm_weight, eps, static_cast<TO*>(out), ld_out, rows, width, streams);                                                 \
+                   norm_weight, eps, static_cast<TO*>(out), ld_out, rows, width, streams, pieces);                                                 \
     } while (0)
 #define MLR_PICK(TO, S)                  \
     do {                                 \
@@ -221,6 +235,25 @@ MLR_API int mlr_streams_step(float* h, const float* y, long long ld_y, const flo
 #undef MLR_PICK
 #undef MLR_GO
     return mlr_launched("streams_step");
+}
+}  // namespace
+
+MLR_API int mlr_streams_step(float* h, const float* y, long long ld_y, const float* y_scale, const float* mix, const float* w_out,
+                             const float* w_in, const float* norm_weight, float eps, void* out, long long ld_out, int out_bf16,
+                             const int* rows, int count, int width, int streams, cudaStream_t stream) {
+    return streams_step(h, y, ld_y, y_scale, mix, w_out, w_in, norm_weight, eps, out, ld_out, out_bf16, rows, count, width, streams, Pieces{}, stream);
+}
+
+// The same with the sub-layer's result given in pieces (`Pieces`: what routed experts leave), added up here.
+MLR_API int mlr_streams_step_pieces(float* h, const float* y, long long ldy, const int* row_of_pair, const float* weights, int top,
+                                    const float* shared_y, long long ld_shared, const float* gate, const void* x, long long ld_x, int x_bf16,
+                                    const float* identity, const float* y_scale, const float* mix, const float* w_out, const float* w_in,
+                                    const float* norm_weight, float eps, void* out, long long ld_out, int out_bf16, int count, int width,
+                                    int streams, cudaStream_t stream) {
+    MLR_REQUIRE(y, "streams_step_pieces: no pieces");
+    const Pieces pieces = {y, ldy, row_of_pair, weights, top, shared_y, ld_shared, gate, x, ld_x, x_bf16, identity};
+    return streams_step(h, nullptr, 0, y_scale, mix, w_out, w_in, norm_weight, eps, out, ld_out, out_bf16, nullptr, count, width, streams, pieces,
+                        stream);
 }
 
 // pairs: [buckets + 1, width] or null (then no state is touched).  state: int32, one value per request slot, `state_stride` apart.

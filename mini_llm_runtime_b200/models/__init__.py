@@ -1,2 +1,2 @@
 """Importing this package registers the architectures."""
-from . import gelulix, gopevik, niridra, qwen3, sokolorn, sopetar  # noqa: F401
+from . import gelulix, gopevik, niridra, qwen3, repolix, sokolorn, sopetar  # noqa: F401

@@ -92,8 +92,8 @@ _SIGNATURES = {
                               c_int, c_float, c_int, c_void_p],
         "mlr_group_rmsnorm_sum": [c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                   c_int, c_float, c_int, c_void_p],
-        "mlr_group_rmsnorm_pieces": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
-                                     c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
+        "mlr_group_rmsnorm_pieces": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p,
+                                     c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
     },
     "layernorm": {
         "mlr_depth_norm": [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_void_p,
@@ -116,14 +116,22 @@ _SIGNATURES = {
                                   c_int, c_int, c_void_p, c_void_p, c_void_p],
         "mlr_linear_recurrence_split": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p,
                                         c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+    },
+    "short_conv": {
         "mlr_short_conv": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
-                           c_int, c_void_p],
-        "mlr_short_conv_step": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p],
+                           c_int, c_void_p, c_void_p],
+        "mlr_short_conv_step": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p,
+                                c_void_p],
         "mlr_short_conv_state": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p],
+        "mlr_conv_rotate_cache": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p,
+                                  c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     },
     "streams": {
         "mlr_streams_step": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
                              c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
+        "mlr_streams_step_pieces": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p,
+                                    c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_longlong,
+                                    c_int, c_int, c_int, c_int, c_void_p],
         "mlr_embed_hashed": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int,
                              c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p],
     },
@@ -137,8 +145,8 @@ _SIGNATURES = {
                                  c_int, c_void_p, c_void_p],
     },
     "experts": {
-        "mlr_experts_route": [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                              c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+        "mlr_experts_route": [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                              c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
         "mlr_experts_arrange": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                 c_void_p],
         "mlr_experts_tensor_cores": [c_int, c_longlong],
@@ -147,8 +155,8 @@ _SIGNATURES = {
         "mlr_experts_max_tiles": [c_int, c_int],
         "mlr_experts_product": [c_void_p, c_longlong, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p,
                                 c_longlong, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p],
-        "mlr_experts_combine": [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int, c_void_p, c_void_p,
-                                c_longlong, c_int, c_int, c_void_p],
+        "mlr_experts_combine": [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_int,
+                                c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p],
     },
     "weights": {
         "mlr_normal_fill": [c_void_p, c_int, c_longlong, c_ulonglong, c_double, c_int, c_void_p],

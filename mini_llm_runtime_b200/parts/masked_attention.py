@@ -228,7 +228,8 @@ def emit_masked_attention(b, desc: MaskedAttentionSpec, q, gate, act, run: RunCo
     table, stride = b.table(run.group), b.table_stride(run.group)
     args = (address(desc), proj.ptr, proj.ld, gate.ptr if gate else None, gate.ld if gate else 0, act.ptr, act.ld)
     where = (run.cache.data_ptr(), run.cache.shape[0])
-    tiled = (proj.dtype is torch.bfloat16 and native.module("attention_masked").mlr_attention_masked_tiles_fit(dim, vdim)
+    maps = max(desc.maps, 1)
+    tiled = (proj.dtype is torch.bfloat16 and dim % 16 == 0 and native.module("attention_masked").mlr_attention_masked_tiles_fit(maps * dim, vdim)
              and act.ld % 2 == 0 and act.ptr % 4 == 0)
     if not tiled:
         # One block per (row, head): the float32 path, and sizes the tiled kernel does not take.

@@ -139,12 +139,11 @@ class GroupRmsNorm(Norm):
         bias = getattr(delta, "bias", None)
         w_pre = then.weight.data_ptr() if out is not None and not plain else None
         if delta.pieces is not None:
-            y, row_of_pair, weights, top, shared, gate = delta.pieces
+            from .experts import piece_arguments
+            y, shared = delta.pieces[0], delta.pieces[4]
             if sum_with is not None or bias is not None or y.dtype is not torch.float32 or (shared is not None and shared.dtype is not torch.float32):
                 raise native.KernelError("the grouped norm adds up float32 pieces without a bias, and not into a sum that it norms")
-            b.launch("norm_grouped", "mlr_group_rmsnorm_pieces", h.ptr, y.ptr, self.width, row_of_pair.ptr, weights.ptr, top,
-                     shared.ptr if shared is not None else None, shared.ld if shared is not None else 0, gate.ptr if gate is not None else None,
-                     self.weight.data_ptr(), w_pre, out.ptr if out is not None else None, out.ld if out is not None else 0,
+            b.launch("norm_grouped", "mlr_group_rmsnorm_pieces", h.ptr, *piece_arguments(delta.pieces, self.width), self.weight.data_ptr(), w_pre, out.ptr if out is not None else None, out.ld if out is not None else 0,
                      int(b.rt.is_bf16), h.rows, self.width, self.groups, self.eps, 1 | (2 if plain else 0), b.stream)
         elif sum_with is not None:
             b.launch("norm_grouped", "mlr_group_rmsnorm_sum", h.ptr, float(sum_with), delta.ptr, delta.ld,

@@ -1,6 +1,6 @@
 """Mixers with a matrix state per head and request (linear attention): retention with a fixed decay
-per head, gated linear attention with a decay per key channel, and the gated delta rule behind short convolutions with a decay per
-head or per key channel.  All are the kernel `mlr_linear_recurrence` (csrc/kernels/recurrence.cu) under different descriptions.
+per head, gated linear attention with a decay per key channel, the gated delta rule behind short convolutions with a decay per
+head or per key channel, and the state-space duality mixer.  All are the kernel `mlr_linear_recurrence` (csrc/kernels/recurrence.cu) under different descriptions.
 
 Retention:   q, k [H, D], v [H, Dv];  q, k rotated on their first values;  k *= D^(-1/2);
              S <- decay_h S + k v^T;  o = S^T q;  o / rms(o) per head, times silu(g);  result = o Wo^T.
@@ -34,9 +34,9 @@ def emit_recurrence(b, mixer, proj, side, act, run: RunContext) -> None:
     state, info = run.state, b.meta("segment_info")
     d = mixer.desc
     if b.le(proj.rows, b.rt.recurrence_fused_rows):
-        # A read-out that norms all heads of a token together cannot happen in a block that owns one head: the kernel then
+        # A read-out whose norm spans heads of a token cannot happen in a block that owns one head: the kernel then
         # leaves its plain float32 outputs in a buffer and the read-out is a second launch.
-        plain = b.temp(proj.rows, d.heads * d.vdim, torch.float32) if d.norm_all else None
+        plain = b.temp(proj.rows, d.heads * d.vdim, torch.float32) if d.norm_all or d.gate_first else None
         b.launch("recurrence", "mlr_linear_recurrence", address(d), proj.ptr, proj.ld, side.ptr, side.ld, proj.is_bf16,
                  act.ptr, act.ld, state.data_ptr(), state.stride(0), info, b.segments, proj.rows, plain.ptr if plain else None,
                  b.status, b.stream)
@@ -61,6 +61,23 @@ def emit_recurrence(b, mixer, proj, side, act, run: RunContext) -> None:
     b.launch("recurrence", "mlr_linear_recurrence_split", address(d), proj.ptr, proj.ld, side.ptr, side.ld, proj.is_bf16, act.ptr,
              act.ld, state.data_ptr(), state.stride(0), info, b.segments, b.meta("positions"), proj.rows, qf.ptr, kf.ptr, gates.ptr,
              obuf.ptr, df.ptr if df else None, gf.ptr if gf else None, made, b.stream)
+
+
+def emit_short_conv(b, x, taps_weight: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, state_offset: int):
+    """The causal convolution (and SiLU) of the channels `x` into a buffer of its own (a row's other tokens read `x` meanwhile); then
+    the convolution's state, the last taps - 1 inputs of every request from float `state_offset` of its slot on, moves on."""
+    at, stride, info = state.data_ptr() + 4 * state_offset, state.stride(0), b.meta("segment_info")
+    channels, taps = taps_weight.shape
+    shift = bias.data_ptr() if bias is not None else None
+    conv = b.temp(x.rows, channels, x.dtype)
+    if b.le(x.rows, b.rt.recurrence_fused_rows):
+        b.launch("short_conv", "mlr_short_conv_step", x.ptr, x.ld, conv.ptr, conv.ld, x.is_bf16, channels, taps, taps_weight.data_ptr(), at, stride,
+                 info, b.segments, shift, b.stream)
+    else:
+        b.launch("short_conv", "mlr_short_conv", x.ptr, x.ld, conv.ptr, conv.ld, x.is_bf16, channels, taps, taps_weight.data_ptr(), at, stride,
+                 info, b.meta("segment_of_row"), x.rows, shift, b.stream)
+        b.launch("short_conv", "mlr_short_conv_state", x.ptr, x.ld, x.is_bf16, channels, taps, at, stride, info, b.segments, b.stream)
+    return conv
 
 
 def _check_state_size(dim: int, vdim: int) -> None:
@@ -165,7 +182,7 @@ class DeltaRuleMixer(SequenceCore):
                 WeightSpec(w["norm"], (self.vdim,), "vector", ("one_plus_normal", 0.01))]
 
     def kernel_modules(self, dtype) -> List[str]:
-        return ["recurrence"] + F.product_modules(dtype)
+        return ["recurrence", "short_conv"] + F.product_modules(dtype)
 
     def bind_core(self, tensors, rt, out_scale: float) -> None:
         w = self.spec.weights
@@ -191,22 +208,8 @@ class DeltaRuleMixer(SequenceCore):
         """What a form of the rule changes in `desc`."""
 
     def emit_core(self, b, proj, act, run: RunContext) -> None:
-        # q, k, v pass the convolutions into a buffer of their own (a row's other tokens read the
-        # projections' output meanwhile); then the convolutions' state moves on; the recurrence reads q, k, v
-        # from the convolved buffer and b, a and the gate from the projections' output.
-        state = run.state
-        conv_state = state.data_ptr() + 4 * self.matrix_floats
-        stride = state.stride(0)
-        info, of_row = b.meta("segment_info"), b.meta("segment_of_row")
-        conv = b.temp(proj.rows, self.channels, proj.dtype)
-        if b.le(proj.rows, b.rt.recurrence_fused_rows):
-            b.launch("recurrence", "mlr_short_conv_step", proj.ptr, proj.ld, conv.ptr, conv.ld, proj.is_bf16, self.channels, self.taps,
-                     self.taps_weight.data_ptr(), conv_state, stride, info, b.segments, b.stream)
-        else:
-            b.launch("recurrence", "mlr_short_conv", proj.ptr, proj.ld, conv.ptr, conv.ld, proj.is_bf16, self.channels, self.taps,
-                     self.taps_weight.data_ptr(), conv_state, stride, info, of_row, proj.rows, b.stream)
-            b.launch("recurrence", "mlr_short_conv_state", proj.ptr, proj.ld, proj.is_bf16, self.channels, self.taps, conv_state, stride,
-                     info, b.segments, b.stream)
+        # The recurrence reads q, k, v from the convolved buffer and b, a and the gate from the projections' output.
+        conv = emit_short_conv(b, columns_of(proj, 0, self.channels), self.taps_weight, None, run.state, self.matrix_floats)
         emit_recurrence(b, self, conv, proj, act, run)
 
 
@@ -383,3 +386,74 @@ class ChannelDeltaMixer(DeltaRuleMixer):
 
 
 register_part("mixer", "channel_delta", ChannelDeltaMixer)
+
+
+class StateSpaceMixer(SequenceCore):
+    """The state-space duality mixer: a state per head with a step size and a decay per token, keys and queries that groups of heads share.
+
+        z | v | k | q | dt = Win x                   [H Dv | H Dv | G N | G N | H]
+        v, k, q through a causal convolution over time per channel, a bias and silu;   dt <- softplus(dt + dt_bias)
+        S <- exp(-exp(A_log_h) dt) S + dt k v^T [N, Dv];  o = S^T q + D_h v          (head h uses k and q number h // (H/G))
+        o (all heads side by side) times silu(z), each of `norm_groups` equal parts over its own root mean square, times a weight [H Dv];
+        result = o Wo^T
+
+    Parameters: hidden_size, num_heads, num_groups (G), state_dim (N), value_dim (Dv), conv (taps), norm_groups, eps.  Weights: "in"
+    [2 H Dv + 2 G N + H, W], "conv" [H Dv + 2 G N, taps], "conv_bias" [H Dv + 2 G N], "dt_bias", "A_log", "D" [H], "norm" [H Dv],
+    "o" [W, H Dv].  The state is float32 [H, Dv, N] per request, followed by the last taps-1 inputs of the convolution."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        p = spec.params
+        self.width = int(p["hidden_size"])
+        self.heads, self.groups = int(p["num_heads"]), int(p["num_groups"])
+        self.dim, self.vdim, self.taps = int(p["state_dim"]), int(p["value_dim"]), int(p["conv"])
+        self.norm_groups, self.eps = int(p["norm_groups"]), float(p["eps"])
+        self.inner = self.heads * self.vdim
+        if self.heads % self.groups:
+            raise ConfigError(f"{self.heads} heads cannot share {self.groups} keys and queries")
+        if self.norm_groups < 1 or self.inner % self.norm_groups:
+            raise ConfigError(f"{self.inner} values cannot be normed in {self.norm_groups} equal parts")
+        if not 1 <= self.taps <= 16:
+            raise ConfigError(f"a convolution of {self.taps} taps is outside what the kernel takes (1 to 16)")
+        _check_state_size(self.dim, self.vdim)
+        self.channels = self.inner + 2 * self.groups * self.dim
+        self.matrix_floats = self.heads * self.vdim * self.dim
+        self.desc: Optional[RecurrenceSpec] = None
+
+    def state_need(self) -> StateNeed:
+        return StateNeed((self.matrix_floats + (self.taps - 1) * self.channels,), torch.float32)
+
+    def in_roles(self) -> List[Tuple[str, int]]:
+        return [("in", self.inner + self.channels + self.heads)]
+
+    def core_width(self) -> int:
+        return self.inner
+
+    def extra_weight_specs(self) -> List[WeightSpec]:
+        w = self.spec.weights
+        vector = lambda role, n, init: WeightSpec(w[role], (n,), "vector", init)
+        return [WeightSpec(w["conv"], (self.channels, self.taps), "vector", ("normal", 0.3)), vector("conv_bias", self.channels, ("normal", 0.1)),
+                vector("dt_bias", self.heads, ("normal", 0.5)), vector("A_log", self.heads, ("normal", 0.5)),
+                vector("D", self.heads, ("one_plus_normal", 0.1)), vector("norm", self.inner, ("one_plus_normal", 0.01))]
+
+    def kernel_modules(self, dtype) -> List[str]:
+        return ["recurrence", "short_conv"] + F.product_modules(dtype)
+
+    def bind_core(self, tensors, rt, out_scale: float) -> None:
+        w = self.spec.weights
+        vec = lambda role: rt.vector(tensors[w[role]]).float().contiguous()
+        self.taps_weight, self.conv_bias = vec("conv"), vec("conv_bias")
+        self._held = {role: vec(role) for role in ("A_log", "dt_bias", "D", "norm")}
+        at = lambda role: self._held[role].data_ptr()
+        self.desc = RecurrenceSpec(
+            a_log=at("A_log"), dt_bias=at("dt_bias"), skip=at("D"), out_weight=at("norm"), heads=self.heads, qk_heads=self.groups, dim=self.dim,
+            vdim=self.vdim, prep=RecurrenceSpec.PREP[None], rot_dims=0, rule=RecurrenceSpec.RULE["step"], gate_kind=GATES["silu"],
+            col_v=0, col_k=self.inner, col_q=self.inner + self.groups * self.dim, col_gate=0, col_a=self.inner + self.channels, gate_first=1,
+            norm_parts=self.norm_groups, q_mult=1.0, k_mult=1.0, unit_eps=0.0, eps=self.eps, out_scale=float(out_scale))
+
+    def emit_core(self, b, proj, act, run: RunContext) -> None:
+        conv = emit_short_conv(b, columns_of(proj, self.inner, self.channels), self.taps_weight, self.conv_bias, run.state, self.matrix_floats)
+        emit_recurrence(b, self, conv, proj, act, run)
+
+
+register_part("mixer", "state_space", StateSpaceMixer)

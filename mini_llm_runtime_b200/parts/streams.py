@@ -23,6 +23,7 @@ from ..config.registry import register_part
 from ..ops import native
 from ..weights.loader import WeightSpec
 from .base import Block, Embedding, Norm, StateNeed
+from .experts import piece_arguments
 
 MAX_STREAMS = 16
 
@@ -131,12 +132,16 @@ class StreamsBlock(Block):
         norm = then.norms["pre_mixer" if then_q == 1 else "pre_feed_forward"] if then is not None else None
         if y is not None and (y.slices or y.norm is not None or y.dtype is not torch.float32):
             raise native.KernelError("a sub-layer of a streams block hands over a plain float32 [rows, width] result")
-        b.launch("streams", "mlr_streams_step", h.ptr, y.ptr if y is not None else None, y.ld if y is not None else 0,
-                 self.w[f"scale{q}"].data_ptr() if y is not None else None, self.w[f"mix{q}"].data_ptr() if y is not None else None,
-                 self.w[f"out{q}"].data_ptr() if y is not None else None, then.w[f"in{then_q}"].data_ptr() if then is not None else None,
-                 then.w[f"norm{then_q}"].data_ptr() if then is not None else None, float(norm.eps) if norm is not None else 0.0,
-                 out.ptr if out is not None else None, out.ld if out is not None else 0, int(b.rt.is_bf16), None, h.rows, self.width,
-                 self.streams, b.stream)
+        at = lambda role: self.w[f"{role}{q}"].data_ptr() if y is not None else None
+        weights = (at("scale"), at("mix"), at("out"), then.w[f"in{then_q}"].data_ptr() if then is not None else None,
+                   then.w[f"norm{then_q}"].data_ptr() if then is not None else None, float(norm.eps) if norm is not None else 0.0,
+                   out.ptr if out is not None else None, out.ld if out is not None else 0, int(b.rt.is_bf16))
+        if y is not None and y.pieces is not None:      # routed experts' results, added up by this launch
+            b.launch("streams", "mlr_streams_step_pieces", h.ptr, *piece_arguments(y.pieces, self.width), *weights, h.rows, self.width, self.streams,
+                     b.stream)
+        else:
+            b.launch("streams", "mlr_streams_step", h.ptr, y.ptr if y is not None else None, y.ld if y is not None else 0, *weights, None, h.rows,
+                     self.width, self.streams, b.stream)
         return out
 
     def forward(self, h, pending, step, run):
@@ -162,7 +167,11 @@ class StreamsBlock(Block):
             ahead = self._step(b, h, mixed, 1, following)
         else:
             x = self._step(b, h, mixed, 1, self, 2)
-            out = self.feed_forward.emit(b, x)
+            b.accepts_pieces = True
+            try:
+                out = self.feed_forward.emit(b, x)
+            finally:
+                b.accepts_pieces = False
             ahead = self._step(b, h, out, 2, following)
         b.prepared = {"streams": following, "stream": h, "out": ahead} if following is not None else None
         return None

@@ -444,9 +444,9 @@ def test_short_convolution_over_steps_of_any_size(taps):
         x = torch.cat([xs[0][at:at + n], xs[1][at:at + n]]).to(dev)
         _, of_row, info = _meta([(0, n, at, slots[0]), (n, n, at, slots[1])], dev)
         out = torch.empty_like(x)
-        _call("recurrence", "mlr_short_conv", x.data_ptr(), channels, out.data_ptr(), channels, 0, channels, taps, weights.data_ptr(),
-              conv_state, per_slot, info.data_ptr(), of_row.data_ptr(), 2 * n, native.stream())
-        _call("recurrence", "mlr_short_conv_state", x.data_ptr(), channels, 0, channels, taps, conv_state, per_slot, info.data_ptr(), 2,
+        _call("short_conv", "mlr_short_conv", x.data_ptr(), channels, out.data_ptr(), channels, 0, channels, taps, weights.data_ptr(),
+              conv_state, per_slot, info.data_ptr(), of_row.data_ptr(), 2 * n, None, native.stream())
+        _call("short_conv", "mlr_short_conv_state", x.data_ptr(), channels, 0, channels, taps, conv_state, per_slot, info.data_ptr(), 2,
               native.stream())
         outs[0].append(out[:n].cpu())
         outs[1].append(out[n:].cpu())

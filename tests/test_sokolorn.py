@@ -188,7 +188,8 @@ def test_norm_behind_routed_experts_adds_up_their_pieces(rows, width, top, share
     hd, yd, rd, wd, od, gd, weight = (t.to(dev) for t in (h, y, row_of_pair, weights, other, gate, w + 1.0))
     out = torch.full((rows, width), float("nan"), dtype=torch.bfloat16, device=dev)
     _call("norm_grouped", "mlr_group_rmsnorm_pieces", hd.data_ptr(), yd.data_ptr(), width, rd.data_ptr(), wd.data_ptr(), top,
-          od.data_ptr() if shared else None, od.stride(0) if shared else 0, gd.data_ptr() if shared and gated else None, weight.data_ptr(), None,
+          od.data_ptr() if shared else None, od.stride(0) if shared else 0, gd.data_ptr() if shared and gated else None, None, 0, 0, None,
+          weight.data_ptr(), None,
           out.data_ptr(), out.stride(0), 1, rows, width, 1, 1e-6, 3, native.stream())
     total = (weights.double()[:, :, None] * y.double()[row_of_pair.long()]).sum(dim=1)
     if shared:
