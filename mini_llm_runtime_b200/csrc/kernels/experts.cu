@@ -69,57 +69,77 @@ __device__ __forceinline__ int warp_argmax(const float* values, int n) {
     return at == INT_MAX ? 0 : at;
 }
 
-template <typename T>
+// ROWS tokens a block: the router's matrix is read once for them; then warp r chooses for the block's token r.
+template <typename T, int ROWS>
 __global__ void __launch_bounds__(kRouteThreads) route_kernel(const T* x, long long ld, const float* router, const float* correction,
-                                                              int width, int experts, int routed, int groups, int keep, int top, int has_gate,
-                                                              int* chosen, float* weights, int* place, int* counts, float* shared_gate,
+                                                              int rows, int width, int experts, int routed, int groups, int keep, int top,
+                                                              int has_gate, int* chosen, float* weights, int* place, int* counts, float* shared_gate,
                                                               float* identity, int kind) {
     mlr_grid_wait();
     extern __shared__ __align__(16) float shared[];
-    float* xs = shared;                 // [width]
-    float* score = xs + width;          // [experts] plain scores
-    float* choice = score + experts;    // [experts] scores with the correction (minus infinity where not allowed, NaN once taken)
-    float* group_score = choice + experts;   // [groups]
-    const int row = blockIdx.x;
+    float* xs = shared;                                 // [ROWS][width]
+    float* scores = xs + static_cast<size_t>(ROWS) * width;   // per row: [experts] plain scores,
+    const int per_row = 2 * experts + groups;           // [experts] scores with the correction (minus infinity where not allowed, NaN once taken),
+                                                        // [groups]
+    const int row0 = blockIdx.x * ROWS;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-    const T* xrow = x + static_cast<size_t>(row) * ld;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) xs[c] = mlr_load(xrow, c);
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+        const T* xrow = x + static_cast<size_t>(min(row0 + r, rows - 1)) * ld;
+        for (int c = threadIdx.x; c < width; c += blockDim.x) xs[static_cast<size_t>(r) * width + c] = mlr_load(xrow, c);
+    }
     __syncthreads();
     for (int e = warp; e < experts + has_gate; e += warps) {
         const float* w = router + static_cast<size_t>(e) * width;
-        float sum = 0.0f;
-        if (width % 4 == 0) {         // 16 bytes at a time (rows of the router and the shared row start on 16-byte borders then)
+        float sums[ROWS] = {};
+        if (width % 4 == 0) {         // 16 bytes at a time (rows of the router and the shared rows start on 16-byte borders then)
             const float4* w4 = reinterpret_cast<const float4*>(w);
             const float4* x4 = reinterpret_cast<const float4*>(xs);
 #pragma unroll 4
             for (int c = lane; c < width / 4; c += 32) {
-                const float4 a = w4[c], b = x4[c];
-                sum = fmaf(a.x, b.x, sum);
-                sum = fmaf(a.y, b.y, sum);
-                sum = fmaf(a.z, b.z, sum);
-                sum = fmaf(a.w, b.w, sum);
+                const float4 a = w4[c];
+#pragma unroll
+                for (int r = 0; r < ROWS; ++r) {
+                    const float4 b = x4[r * (width / 4) + c];
+                    sums[r] = fmaf(a.x, b.x, sums[r]);
+                    sums[r] = fmaf(a.y, b.y, sums[r]);
+                    sums[r] = fmaf(a.z, b.z, sums[r]);
+                    sums[r] = fmaf(a.w, b.w, sums[r]);
+                }
             }
         } else {
-            for (int c = lane; c < width; c += 32) sum = fmaf(w[c], xs[c], sum);
+            for (int c = lane; c < width; c += 32) {
+#pragma unroll
+                for (int r = 0; r < ROWS; ++r) sums[r] = fmaf(w[c], xs[static_cast<size_t>(r) * width + c], sums[r]);
+            }
         }
-        sum = mlr_warp_sum(sum);
-        if (lane == 0) {
-            if (e >= experts) {
-                shared_gate[row] = 1.0f / (1.0f + expf(-sum));
-            } else if (kind == 2) {
-                score[e] = sum;
-            } else if (kind == 1) {
-                score[e] = choice[e] = sum + (correction ? correction[e] : 0.0f);
-            } else {
-                const float s = 1.0f / (1.0f + expf(-sum));
-                score[e] = s;
-                choice[e] = s + (correction ? correction[e] : 0.0f);
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            const float sum = mlr_warp_sum(sums[r]);
+            float* score = scores + static_cast<size_t>(r) * per_row;
+            float* choice = score + experts;
+            if (lane == 0 && row0 + r < rows) {
+                if (e >= experts) {
+                    shared_gate[row0 + r] = 1.0f / (1.0f + expf(-sum));
+                } else if (kind == 2) {
+                    score[e] = sum;
+                } else if (kind == 1) {
+                    score[e] = choice[e] = sum + (correction ? correction[e] : 0.0f);
+                } else {
+                    const float s = 1.0f / (1.0f + expf(-sum));
+                    score[e] = s;
+                    choice[e] = s + (correction ? correction[e] : 0.0f);
+                }
             }
         }
     }
     __syncthreads();
-    if (warp != 0) return;
-    // One warp chooses.
+    if (warp >= ROWS || row0 + warp >= rows) return;
+    // One warp chooses for a token.
+    const int row = row0 + warp;
+    float* score = scores + static_cast<size_t>(warp) * per_row;
+    float* choice = score + experts;
+    float* group_score = choice + experts;
     if (kind == 2) {
         float largest = -INFINITY, total = 0.0f;
         for (int e = lane; e < experts; e += 32) largest = fmaxf(largest, score[e]);
@@ -481,19 +501,27 @@ MLR_API int mlr_experts_route(const void* x, long long ld, int act_bf16, const f
                 "experts_route: %d experts in %d groups of which %d are kept cannot give %d", experts, groups, keep, top);
     MLR_REQUIRE(!has_gate || shared_gate, "experts_route: no room for the shared expert's gate");
     if (rows <= 0) return 0;
-    const size_t shared = sizeof(float) * (static_cast<size_t>(width) + 2 * experts + groups);
-    MLR_REQUIRE(shared <= 200 * 1024, "experts_route: a row of %d values and %d experts do not fit shared memory", width, experts);
-    // Few rows: few blocks, each with a warp per expert.  Many rows: the SMs are full anyway, and smaller blocks waste fewer warps.
+    // Few rows: few blocks, each with a warp per expert.  Many rows: the SMs are full anyway, smaller blocks waste fewer warps, and four tokens
+    // a block share the reading of the router's matrix.
+    const size_t one = sizeof(float) * (static_cast<size_t>(width) + 2 * experts + groups);
+    MLR_REQUIRE(one <= 200 * 1024, "experts_route: a row of %d values and %d experts do not fit shared memory", width, experts);
+    const int per_block = rows >= 4 * 148 && 4 * one <= 100 * 1024 ? 4 : 1;
+    const size_t shared = per_block * one;
     const int threads = rows <= 64 ? kRouteThreads : 256;
+#define MLR_ROUTE(T, ROWS)                                                                                                             \
+    do {                                                                                                                               \
+        if (shared > 48 * 1024) cudaFuncSetAttribute(route_kernel<T, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared)); \
+        mlr_launch((route_kernel<T, ROWS>), dim3((rows + ROWS - 1) / ROWS), dim3(threads), shared, stream, static_cast<const T*>(x), ld, router, \
+                   correction, rows, width, experts, routed, groups, keep, top, has_gate, chosen, weights, place, counts, shared_gate, identity, kind); \
+    } while (0)
     if (act_bf16) {
-        if (shared > 48 * 1024) cudaFuncSetAttribute(route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));
-        mlr_launch((route_kernel<__nv_bfloat16>), dim3(rows), dim3(threads), shared, stream, static_cast<const __nv_bfloat16*>(x), ld, router,
-                   correction, width, experts, routed, groups, keep, top, has_gate, chosen, weights, place, counts, shared_gate, identity, kind);
+        if (per_block == 4) MLR_ROUTE(__nv_bfloat16, 4);
+        else MLR_ROUTE(__nv_bfloat16, 1);
     } else {
-        if (shared > 48 * 1024) cudaFuncSetAttribute(route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));
-        mlr_launch((route_kernel<float>), dim3(rows), dim3(threads), shared, stream, static_cast<const float*>(x), ld, router, correction, width,
-                   experts, routed, groups, keep, top, has_gate, chosen, weights, place, counts, shared_gate, identity, kind);
+        if (per_block == 4) MLR_ROUTE(float, 4);
+        else MLR_ROUTE(float, 1);
     }
+#undef MLR_ROUTE
     return mlr_launched("experts_route");
 }
 

@@ -82,16 +82,17 @@ __global__ void __launch_bounds__(kThreads) streams_step_kernel(float* h, const 
         if (writes) {
             float add[V];
             if (yrow) {
-#pragma unroll
-                for (int e = 0; e < V; ++e) add[e] = __ldcg(yrow + c + e);
+                mlr_load_group<V>(yrow + c, add);
             } else {
                 const float4 v = piece_sum<V == 4>(pieces, staged, row, c);
                 add[0] = v.x;
                 if (V == 4) add[V > 1 ? 1 : 0] = v.y, add[V > 2 ? 2 : 0] = v.z, add[V - 1] = v.w;
             }
             if (y_scale) {
+                float scale[V];
+                mlr_load_group<V>(y_scale + c, scale);
 #pragma unroll
-                for (int e = 0; e < V; ++e) add[e] *= y_scale[c + e];
+                for (int e = 0; e < V; ++e) add[e] *= scale[e];
             }
 #pragma unroll
             for (int t = 0; t < kCopies; ++t) {
@@ -139,7 +140,13 @@ __global__ void __launch_bounds__(kThreads) streams_step_kernel(float* h, const 
     }
     const float inv = 1.0f / sqrtf(mlr_block_sum(squares, scratch) / static_cast<float>(width) + eps);
     TO* orow = out + static_cast<size_t>(blockIdx.x) * ld_out;
-    for (int c = threadIdx.x; c < width; c += kThreads) mlr_store(orow, c, u[c] * inv * (norm_weight ? norm_weight[c] : 1.0f));
+    for (int c = threadIdx.x * V; c < width; c += kThreads * V) {         // a thread's own columns
+        float value[V], weight[V];
+        if (norm_weight) mlr_load_group<V>(norm_weight + c, weight);
+#pragma unroll
+        for (int e = 0; e < V; ++e) value[e] = u[c + e] * inv * (norm_weight ? weight[e] : 1.0f);
+        mlr_store_group<V>(orow + c, value);
+    }
     mlr_grid_dependents_may_start();
 }
 
@@ -205,7 +212,9 @@ int streams_step(float* h, const float* y, long long ld_y, const float* y_scale,
     MLR_REQUIRE(static_cast<size_t>(width) * sizeof(float) <= 200 * 1024, "streams_step: a width of %d does not fit shared memory", width);
     if (count <= 0) return 0;
     const size_t shared = out ? static_cast<size_t>(width) * sizeof(float) : 0;
-    const bool wide = width % 4 == 0 && reinterpret_cast<uintptr_t>(h) % 16 == 0 && (!pieces.y || pieces_aligned(pieces));
+    const auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    const bool wide = width % 4 == 0 && aligned(h) && aligned(y) && ld_y % 4 == 0 && aligned(y_scale) && aligned(norm_weight) && aligned(out) &&
+                      ld_out % 4 == 0 && (!pieces.y || pieces_aligned(pieces));
 #define MLR_GO(TO, S, V)                                                                                                                   \
     do {                                                                                                                                   \
         if (shared > 48 * 1024)                                                                                                            \

@@ -313,9 +313,10 @@ def test_recurrences_alone_in_both_forms(dtype, fused, kind, mixer):
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("experts,identity,groups,keep,top", [(6, 3, 3, 2, 3), (5, 0, 1, 1, 2), (12, 4, 4, 3, 4), (1, 7, 2, 1, 3), (64, 16, 8, 3, 8), (3, 2, 5, 2, 2),
                                                               (40, 24, 64, 32, 32), (7, 1, 1, 1, 8)])
-def test_router_with_groups_and_identity_experts(dtype, experts, identity, groups, keep, top):
+@pytest.mark.parametrize("rows,width", [(37, 24), (601, 18)])            # one token a block, and four
+def test_router_with_groups_and_identity_experts(dtype, experts, identity, groups, keep, top, rows, width):
     from mini_llm_runtime_b200.ops import native
-    dev, rows, width = "cuda:0", 37, 24
+    dev = "cuda:0"
     everyone = experts + identity
     g = torch.Generator().manual_seed(everyone)
     x = torch.randn(rows, width, generator=g).to(dtype).to(dev)
@@ -328,7 +329,7 @@ def test_router_with_groups_and_identity_experts(dtype, experts, identity, group
           everyone, experts, groups, keep, top, 0, chosen.data_ptr(), weights.data_ptr(), place.data_ptr(), counts.data_ptr(), None,
           passed.data_ptr() if identity else None, 2, native.stream())
     scores = torch.softmax(x.double().cpu() @ router.double().cpu().T, dim=-1)
-    for t in range(rows):
+    for t in list(range(37)) + list(range(37, rows, 41)) + [rows - 1]:
         want = plain.choose(scores[t], correction.double().cpu(), top, groups, keep)
         assert chosen[t].tolist() == want
         assert torch.allclose(weights[t].double().cpu(), scores[t, want], atol=1e-6)
@@ -343,7 +344,7 @@ def test_router_with_groups_and_identity_experts(dtype, experts, identity, group
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("rows", [1, 3, 70, 300])
+@pytest.mark.parametrize("rows", [1, 3, 70, 700])
 @pytest.mark.parametrize("shape", [(24, 6, 3, (3, 2), 3, 56), (32, 8, 0, None, 2, None), (10, 2, 6, (2, 1), 2, 12)])
 def test_routed_experts_part_against_the_plain_function(dtype, rows, shape):
     """The part by hand, run twice: counters return to zero, tokens whose experts are all identity experts among them."""
