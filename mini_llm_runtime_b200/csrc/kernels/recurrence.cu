@@ -650,39 +650,43 @@ __global__ void __launch_bounds__(kScanWarps * 32) recurrence_scan_kernel(const 
 // between; a token's k, q and decays are loaded from shared memory while the token before it is walked.
 constexpr int kColumnLanes = 16, kColumnWarps = kScanBlockCols * kColumnLanes / 32;
 
-template <typename T, int DIM, int RULE, bool CH>
+// NC: columns of the state a lane works on (column c and c + 16): two halve the reading of k and q where blocks outnumber the SMs.
+template <typename T, int DIM, int RULE, bool CH, int NC>
 __global__ void __launch_bounds__(kColumnWarps * 32) recurrence_scan16_kernel(const float* qf, const float* kf, const float* df, const float* gates,
                                                                             const T* proj, int ld, float* obuf, float* state, long long state_stride,
                                                                             const int* segment_info, RecurrenceSpec s, int batch) {
     mlr_grid_wait();
     constexpr int kThreads = kColumnWarps * 32, E = DIM / kColumnLanes, V = E % 4 == 0 ? 4 : 2;       // V: values an access
+    constexpr int kCols = kScanBlockCols * NC;
     extern __shared__ __align__(16) unsigned char smem[];
     const int stage = batch * DIM;                             // batch: a multiple of 4, at most 32
     float* qs = reinterpret_cast<float*>(smem);                // [2][batch][DIM]: a batch is copied while the one before is walked
     float* ks = qs + 2 * stage;                                // [2][batch][DIM]
     float* ds = ks + 2 * stage;                                // CH: [2][batch][DIM], decays per channel
-    float* vs = ds + (CH ? 2 * stage : 0);                     // [16][batch]
-    float* os = vs + batch * kScanBlockCols;                   // [batch][16]
-    float* gs = os + batch * kScanBlockCols;                   // [batch]
+    float* vs = ds + (CH ? 2 * stage : 0);                     // [kCols][batch]
+    float* os = vs + batch * kCols;                   // [batch][kCols]
+    float* gs = os + batch * kCols;                   // [batch]
     float* bs = gs + batch;                                    // [batch]
-    const int segment = blockIdx.x, head = blockIdx.y, block_col = blockIdx.z * kScanBlockCols;
+    const int segment = blockIdx.x, head = blockIdx.y, block_col = blockIdx.z * kCols;
     const int first = segment_info[4 * segment], count = segment_info[4 * segment + 1], slot = segment_info[4 * segment + 3];
     const int qk_head = head / (s.heads / s.qk_heads);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int sub = lane & (kColumnLanes - 1), my_col = warp * (32 / kColumnLanes) + lane / kColumnLanes;
-    const bool live = block_col + my_col < s.vdim;
     const size_t qk_ld = static_cast<size_t>(s.qk_heads) * DIM, d_ld = static_cast<size_t>(s.heads) * DIM;
     const size_t o_ld = static_cast<size_t>(s.heads) * s.vdim;
     const float decay = !CH && RULE == 0 ? s.decay[head] : 1.0f;
 
-    float S[E];
+    float S[NC][E];
     float* my_state = state + static_cast<size_t>(slot) * state_stride + (static_cast<size_t>(head) * s.vdim + block_col + my_col) * DIM;
+    auto live = [&](int n) { return block_col + my_col + n * kScanBlockCols < s.vdim; };
     // Value j of a lane is value V * (16 * (j / V) + sub) + j % V of the head: sixteen lanes read consecutive bytes.
     auto place = [&](int j) { return V * (kColumnLanes * (j / V) + sub) + j % V; };
 #pragma unroll
-    for (int j = 0; j < E; ++j) S[j] = live ? my_state[place(j)] : 0.0f;
+    for (int n = 0; n < NC; ++n)
+#pragma unroll
+        for (int j = 0; j < E; ++j) S[n][j] = live(n) ? my_state[n * kScanBlockCols * DIM + place(j)] : 0.0f;
 
-    constexpr int kVPerThread = 32 * kScanBlockCols / kThreads;
+    constexpr int kVPerThread = 32 * kCols / kThreads;
     T v_next[kVPerThread];                // as loaded: a conversion right behind the load would wait for it
     float g_next = 0.0f, b_next = 0.0f;
     // Starts the copies of a batch's q, k and decays into a stage and loads its v, g and beta into registers.
@@ -705,7 +709,7 @@ __global__ void __launch_bounds__(kColumnWarps * 32) recurrence_scan16_kernel(co
 #pragma unroll
         for (int j = 0; j < kVPerThread; ++j) {
             const int i = threadIdx.x + j * kThreads;
-            const int t = i / kScanBlockCols, c = block_col + i % kScanBlockCols;
+            const int t = i / kCols, c = block_col + i % kCols;
             v_next[j] = proj[(t < n && c < s.vdim) ? static_cast<size_t>(first + base + t) * ld + s.col_v + head * s.vdim + c : 0];
         }
         if (RULE != 0 && threadIdx.x < n) {
@@ -726,7 +730,7 @@ __global__ void __launch_bounds__(kColumnWarps * 32) recurrence_scan16_kernel(co
 #pragma unroll
         for (int j = 0; j < kVPerThread; ++j) {
             const int i = threadIdx.x + j * kThreads;
-            if (i < batch * kScanBlockCols) vs[i % kScanBlockCols * batch + i / kScanBlockCols] = act_in(mlr_load(&v_next[j], 0), s.in_act);
+            if (i < batch * kCols) vs[i % kCols * batch + i / kCols] = act_in(mlr_load(&v_next[j], 0), s.in_act);
         }
         if (RULE != 0 && threadIdx.x < batch) {
             gs[threadIdx.x] = g_next;
@@ -760,8 +764,12 @@ __global__ void __launch_bounds__(kColumnWarps * 32) recurrence_scan16_kernel(co
         // GUARDED: the batch's last, incomplete group of four.  Rows past the batch are not read: a token's successor is at most the last.
         auto walk4 = [&](int t0, auto guarded) {
             constexpr bool kGuarded = decltype(guarded)::value;
-            const float4 v4 = *reinterpret_cast<const float4*>(vs + my_col * batch + t0);
-            const float v[4] = {v4.x, v4.y, v4.z, v4.w};
+            float v[NC][4];
+#pragma unroll
+            for (int m = 0; m < NC; ++m) {
+                const float4 v4 = *reinterpret_cast<const float4*>(vs + (my_col + m * kScanBlockCols) * batch + t0);
+                v[m][0] = v4.x; v[m][1] = v4.y; v[m][2] = v4.z; v[m][3] = v4.w;
+            }
             [[maybe_unused]] float g[4] = {decay, decay, decay, decay}, beta[4] = {};
             if constexpr (RULE != 0) {
                 const float4 b4 = *reinterpret_cast<const float4*>(bs + t0);
@@ -771,62 +779,71 @@ __global__ void __launch_bounds__(kColumnWarps * 32) recurrence_scan16_kernel(co
                     g[0] = g4.x; g[1] = g4.y; g[2] = g4.z; g[3] = g4.w;
                 }
             }
-            float dots[4];
+            float dots[NC][4];
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
-                dots[u] = 0.0f;
+#pragma unroll
+                for (int m = 0; m < NC; ++m) dots[m][u] = 0.0f;
                 if (!kGuarded || t0 + u < n) {
                     const Token& x = tokens[u & 1];
                     load(tokens[(u + 1) & 1], u < 3 && !kGuarded ? t0 + u + 1 : min(t0 + u + 1, n - 1));
-                    float write = RULE == 2 ? beta[u] * v[u] : v[u];
-                    if constexpr (RULE != 1) {
 #pragma unroll
-                        for (int j = 0; j < E; ++j) S[j] = fmaf(CH ? x.d[CH ? j : 0] : g[u], S[j], x.k[j] * write);
-                    } else {
-                        float c[2] = {};
+                    for (int m = 0; m < NC; ++m) {
+                        float write = RULE == 2 ? beta[u] * v[m][u] : v[m][u];
+                        if constexpr (RULE != 1) {
 #pragma unroll
-                        for (int j = 0; j < E; ++j) {
-                            S[j] *= CH ? x.d[CH ? j : 0] : g[u];
-                            c[j & 1] = fmaf(S[j], x.k[j], c[j & 1]);
+                            for (int j = 0; j < E; ++j) S[m][j] = fmaf(CH ? x.d[CH ? j : 0] : g[u], S[m][j], x.k[j] * write);
+                        } else {
+                            float c[2] = {};
+#pragma unroll
+                            for (int j = 0; j < E; ++j) {
+                                S[m][j] *= CH ? x.d[CH ? j : 0] : g[u];
+                                c[j & 1] = fmaf(S[m][j], x.k[j], c[j & 1]);
+                            }
+                            float held = c[0] + c[1];
+#pragma unroll
+                            for (int step = 1; step < kColumnLanes; step *= 2) held += __shfl_xor_sync(0xffffffffu, held, step);
+                            write = beta[u] * (write - held);
+#pragma unroll
+                            for (int j = 0; j < E; ++j) S[m][j] = fmaf(x.k[j], write, S[m][j]);
                         }
-                        float held = c[0] + c[1];
+                        float o[2] = {};
 #pragma unroll
-                        for (int step = 1; step < kColumnLanes; step *= 2) held += __shfl_xor_sync(0xffffffffu, held, step);
-                        write = beta[u] * (write - held);
-#pragma unroll
-                        for (int j = 0; j < E; ++j) S[j] = fmaf(x.k[j], write, S[j]);
+                        for (int j = 0; j < E; ++j) o[j & 1] = fmaf(S[m][j], x.q[j], o[j & 1]);
+                        dots[m][u] = o[0] + o[1];
                     }
-                    float o[2] = {};
-#pragma unroll
-                    for (int j = 0; j < E; ++j) o[j & 1] = fmaf(S[j], x.q[j], o[j & 1]);
-                    dots[u] = o[0] + o[1];
                 }
             }
             // Lanes with sub % 4 == u end up with the sum of token t0 + u.
             const bool odd = sub & 1, high = sub & 2;
-            const float even_pair = (odd ? dots[1] : dots[0]) + __shfl_xor_sync(0xffffffffu, odd ? dots[0] : dots[1], 1);
-            const float odd_pair = (odd ? dots[3] : dots[2]) + __shfl_xor_sync(0xffffffffu, odd ? dots[2] : dots[3], 1);
-            float sum = (high ? odd_pair : even_pair) + __shfl_xor_sync(0xffffffffu, high ? even_pair : odd_pair, 2);
-            sum += __shfl_xor_sync(0xffffffffu, sum, 4);
-            sum += __shfl_xor_sync(0xffffffffu, sum, 8);
-            if (sub < 4 && (!kGuarded || t0 + sub < n)) os[(t0 + sub) * kScanBlockCols + my_col] = sum;
+#pragma unroll
+            for (int m = 0; m < NC; ++m) {
+                const float even_pair = (odd ? dots[m][1] : dots[m][0]) + __shfl_xor_sync(0xffffffffu, odd ? dots[m][0] : dots[m][1], 1);
+                const float odd_pair = (odd ? dots[m][3] : dots[m][2]) + __shfl_xor_sync(0xffffffffu, odd ? dots[m][2] : dots[m][3], 1);
+                float sum = (high ? odd_pair : even_pair) + __shfl_xor_sync(0xffffffffu, high ? even_pair : odd_pair, 2);
+                sum += __shfl_xor_sync(0xffffffffu, sum, 4);
+                sum += __shfl_xor_sync(0xffffffffu, sum, 8);
+                if (sub < 4 && (!kGuarded || t0 + sub < n)) os[(t0 + sub) * kCols + my_col + m * kScanBlockCols] = sum;
+            }
         };
         for (int t0 = 0; t0 < n; t0 += 4) {
             if (t0 + 4 <= n) walk4(t0, std::false_type{});      // whole groups carry no per-token conditions
             else walk4(t0, std::true_type{});
         }
         __syncthreads();
-        for (int i = threadIdx.x; i < n * kScanBlockCols; i += kThreads) {
-            const int t = i / kScanBlockCols, c = block_col + i % kScanBlockCols;
-            const float o = RULE == 2 ? fmaf(s.skip[head], vs[i % kScanBlockCols * batch + t], os[i]) : os[i];
+        for (int i = threadIdx.x; i < n * kCols; i += kThreads) {
+            const int t = i / kCols, c = block_col + i % kCols;
+            const float o = RULE == 2 ? fmaf(s.skip[head], vs[i % kCols * batch + t], os[i]) : os[i];
             if (c < s.vdim) obuf[static_cast<size_t>(first + base + t) * o_ld + static_cast<size_t>(head) * s.vdim + c] = o;
         }
     }
     mlr_grid_dependents_may_start();     // only now: blocks of the next grid that wait on this SM slow the walk
-    if (live) {
 #pragma unroll
-        for (int j = 0; j < E; ++j) my_state[place(j)] = S[j];
-    }
+    for (int n = 0; n < NC; ++n)
+        if (live(n)) {
+#pragma unroll
+            for (int j = 0; j < E; ++j) my_state[n * kScanBlockCols * DIM + place(j)] = S[n][j];
+        }
 }
 
 
@@ -1081,12 +1098,17 @@ MLR_API int mlr_linear_recurrence_split(const RecurrenceSpec* spec, const void* 
     const int regs = s.dim <= 32 ? 1 : s.dim <= 64 ? 2 : s.dim <= 128 ? 4 : 8;
     const bool channel = s.channel_decay != 0;
     // q and k (and the channels' decays) in two stages
-    const size_t per_token = sizeof(float) * ((channel ? 6 : 4) * static_cast<size_t>(s.dim) + 2 * kScanBlockCols + 2);
+    // The step rule's walk takes two state columns a lane where blocks of sixteen columns would outnumber the SMs.
+    const bool fixed_size = s.dim == 32 || s.dim == 64 || s.dim == 96 || s.dim == 128 || s.dim == 256;
+    const int column_blocks = (s.vdim + kScanBlockCols - 1) / kScanBlockCols;
+    const bool two = s.rule == 2 && fixed_size && column_blocks > 1 && static_cast<long long>(n_segments) * s.heads * column_blocks > mlr_sm_count();
+    const int block_cols = kScanBlockCols * (two ? 2 : 1);
+    const size_t per_token = sizeof(float) * ((channel ? 6 : 4) * static_cast<size_t>(s.dim) + 2 * block_cols + 2);
     int batch = static_cast<int>(((channel ? 84 : 44) * 1024) / per_token);
     batch = batch < 1 ? 1 : (batch > 32 ? 32 : batch);
     if (batch > 4) batch -= batch % 4;
     const size_t shared = per_token * batch + (channel ? 16 : 0);
-    const dim3 grid(n_segments, s.heads, (s.vdim + kScanBlockCols - 1) / kScanBlockCols);
+    const dim3 grid(n_segments, s.heads, (s.vdim + block_cols - 1) / block_cols);
     const int group = s.heads * s.dim % 4 == 0 && s.heads * s.vdim % 4 == 0 ? 4 : 1;       // channels a thread of the channel kernel
     const int per_block = kChannelThreads * group;
     const dim3 channel_grid((rows + kChannelRows - 1) / kChannelRows,
@@ -1100,9 +1122,10 @@ MLR_API int mlr_linear_recurrence_split(const RecurrenceSpec* spec, const void* 
     } while (0)
 #define MLR_COLUMN(T, DIM, CH)                                                                                                         \
     do {                                                                                                                               \
-        if (s.rule == 0) MLR_WALK((recurrence_scan16_kernel<T, DIM, 0, CH>), T, kColumnWarps);                                         \
-        else if (s.rule == 2) MLR_WALK((recurrence_scan16_kernel<T, DIM, 2, false>), T, kColumnWarps);                                 \
-        else MLR_WALK((recurrence_scan16_kernel<T, DIM, 1, CH>), T, kColumnWarps);                                                     \
+        if (s.rule == 0) MLR_WALK((recurrence_scan16_kernel<T, DIM, 0, CH, 1>), T, kColumnWarps);                                      \
+        else if (s.rule == 2 && two) MLR_WALK((recurrence_scan16_kernel<T, DIM, 2, false, 2>), T, kColumnWarps);                       \
+        else if (s.rule == 2) MLR_WALK((recurrence_scan16_kernel<T, DIM, 2, false, 1>), T, kColumnWarps);                              \
+        else MLR_WALK((recurrence_scan16_kernel<T, DIM, 1, CH, 1>), T, kColumnWarps);                                                  \
     } while (0)
 #define MLR_SCAN(T, CH)                                                                                                                \
     do {                                                                                                                               \

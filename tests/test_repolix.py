@@ -279,6 +279,7 @@ STATES = [
     ("mamba2", dict(heads=3, groups=3, state=100, vdim=16, conv=7, norm_groups=3)),
     ("mamba2", dict(heads=2, groups=2, state=256, vdim=32, conv=2, norm_groups=8)),
     ("mamba2", dict(heads=1, groups=1, state=96, vdim=160, conv=4, norm_groups=5)),
+    ("mamba2", dict(heads=40, groups=4, state=32, vdim=40, conv=2, norm_groups=10)),       # more blocks than SMs: two state columns a lane
     ("channel_delta", dict(heads=6, kv_heads=2, dim=12, vdim=20, conv=4, decay_rank=7, gate_rank=9)),
     ("channel_delta", dict(heads=2, kv_heads=2, dim=64, vdim=32, conv=3, decay_rank=16, gate_rank=8)),
 ]
