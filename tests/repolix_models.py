@@ -62,7 +62,7 @@ ALL = {
         _state(3, 3, 40, 9, 1, 1, _moe(20, 1.0, 7, 2, groups=(7, 3)))]),
     # Sizes the tensor cores and the wide walk take; a prompt beyond one tile of rows; more maps on a key/value head than one tile of heads.
     "small_c": _model(200, 64, 1e-6, 1.4, [
-        _attention(4, 2, 32, 64, 0.2, 0.5, 3, 70, (16, 5000.0, (4.0, 96, 8.0, 2.0)), _moe(64, 2.0, 16, 8, identity=4, groups=(5, 3), shared=(96, 1.5))),
+        _attention(6, 2, 32, 64, 0.2, 0.5, 3, 70, (16, 5000.0, (4.0, 96, 8.0, 2.0)), _moe(64, 2.0, 16, 8, identity=4, groups=(5, 3), shared=(96, 1.5))),
         _state(4, 2, 64, 32, 4, 4, _moe(32, 1.0, 8, 2, identity=8, groups=(2, 2))),
         _attention(18, 1, 16, 8, 0.3, 0.2, 2, 33, (16, 300.0, (32.0, 16, 1.0, 0.1))),
         _state(2, 1, 128, 16, 2, 2), _attention(2, 2, 64, 96, 0.12, 0.6, 4, None, (64, 1e4, (40.0, 4096, 32.0, 1.0)))]),

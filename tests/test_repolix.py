@@ -204,7 +204,7 @@ def test_convolved_and_rotated_projections(dtype, heads, kv_heads, dim, vdim, ta
             assert torch.allclose(got_v, cv.reshape(T, kv_heads, vdim), atol=5 * tol, rtol=tol)
 
 
-ATTENTIONS = [(2, 1, 16, 16, None), (4, 2, 32, 64, 70), (6, 2, 48, 40, 33), (2, 2, 128, 128, 64), (18, 1, 16, 8, None), (3, 3, 7, 5, 20), (2, 1, 64, 96, 1),
+ATTENTIONS = [(2, 1, 16, 16, None), (8, 2, 32, 64, 70), (6, 2, 48, 40, 33), (2, 2, 128, 128, 64), (18, 1, 16, 8, None), (3, 3, 7, 5, 20), (2, 1, 64, 96, 1),
               (1, 1, 24, 160, 50)]
 HOWS = ["rows", ("tiles", 77), ("split", 1, 64, 4, 1), ("split", 1, 128, 2, 4)]
 
@@ -273,7 +273,7 @@ def _mixer(kind, mixer, width, eps, dtype, seed):
 
 STATES = [
     ("mamba2", dict(heads=3, groups=1, state=10, vdim=7, conv=5, norm_groups=7)),
-    ("mamba2", dict(heads=4, groups=2, state=32, vdim=48, conv=3, norm_groups=1)),
+    ("mamba2", dict(heads=4, groups=2, state=32, vdim=56, conv=3, norm_groups=1)),
     ("mamba2", dict(heads=6, groups=6, state=64, vdim=20, conv=1, norm_groups=4)),
     ("mamba2", dict(heads=2, groups=1, state=128, vdim=64, conv=4, norm_groups=2)),
     ("mamba2", dict(heads=3, groups=3, state=100, vdim=16, conv=7, norm_groups=3)),
@@ -312,7 +312,7 @@ def test_recurrences_alone_in_both_forms(dtype, fused, kind, mixer):
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("experts,identity,groups,keep,top", [(6, 3, 3, 2, 3), (5, 0, 1, 1, 2), (12, 4, 4, 3, 4), (1, 7, 2, 1, 3), (64, 16, 8, 3, 8), (3, 2, 5, 2, 2),
+@pytest.mark.parametrize("experts,identity,groups,keep,top", [(6, 3, 3, 2, 3), (5, 0, 1, 1, 2), (10, 6, 4, 3, 5), (1, 7, 2, 1, 3), (64, 16, 8, 3, 8), (3, 2, 5, 2, 2),
                                                               (40, 24, 64, 32, 32), (7, 1, 1, 1, 8)])
 @pytest.mark.parametrize("rows,width", [(37, 24), (601, 18)])            # one token a block, and four
 def test_router_with_groups_and_identity_experts(dtype, experts, identity, groups, keep, top, rows, width):
